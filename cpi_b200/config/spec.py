@@ -41,6 +41,8 @@ class LayerSpec:
     feed_forward: Optional[PartSpec]   # e.g. kind "dense_swiglu" or "moe_swiglu"; None: the layer has no feed-forward
     mixer_norm: PartSpec
     feed_forward_norm: Optional[PartSpec]
+    mixer_post_norm: Optional[PartSpec] = None          # norms on the sublayers' outputs, for a block that has both
+    feed_forward_post_norm: Optional[PartSpec] = None   # (kind "sandwich_norm")
 
 
 @dataclass(frozen=True)
@@ -63,7 +65,7 @@ class ModelSpec:
     architecture: str
     hidden_size: int
     vocab_size: int
-    embedding: PartSpec            # kind "token_embedding", params: weight name
+    embedding: PartSpec            # kind "token_embedding", params: weight name, optional scale (rows are multiplied by it)
     layers: tuple                  # of LayerSpec
     run_order: tuple               # of RunEntry
     final_norm: PartSpec

@@ -255,6 +255,7 @@ struct QkvPrepParams {
   int v_from_k;                          // the values are the k rows as projected (bias added, before any norm); rows hold no v
   int temperature; float floor_scale; float attn_scale;      // q *= 1 + attn_scale * ln(floor((pos + 1) / floor_scale) + 1)
   float rot_amp;                         // the sines and cosines of the rotation are multiplied by this
+  const float* v_inv_freq;               // [DV / 2] or null: values turn over all their elements by these frequencies
 };
 
 // which element a rotated element d is paired with, whether it is the pair's first, and the pair's frequency index
@@ -410,14 +411,21 @@ __global__ void __launch_bounds__(1024) qkv_prepare_kernel(QkvPrepParams p) {
     if (is_q) store_q(i, x);
     else store_k(e, x);
   }
+  const int v_src = p.v_from_k ? nq : nq + nk;             // v_from_k: the key as projected, its bias added, before the norm
+  auto value = [&](int i) {
+    float x = to_f32(src[v_src + i]);
+    if (p.bias) x += load_any(p.bias, p.bias_dtype, v_src + i);
+    return x;
+  };
   for (int i = v0 + tid; i < v1; i += blockDim.x) {
-    float x;
-    if (p.v_from_k) {                                    // the key as projected, its bias added, before the norm
-      x = to_f32(src[nq + i]);
-      if (p.bias) x += load_any(p.bias, p.bias_dtype, nq + i);
-    } else {
-      x = to_f32(src[nq + nk + i]);
-      if (p.bias) x += load_any(p.bias, p.bias_dtype, nq + nk + i);
+    float x = value(i);
+    if (p.v_inv_freq) {
+      bool first; int od, f;
+      rot_pair(i % DV, DV >> 1, p.interleaved, first, od, f);
+      const float other = value(i - i % DV + od);
+      float sn, cs;
+      sincosf((float)pos * p.v_inv_freq[f], &sn, &cs);
+      x = first ? x * cs - other * sn : x * cs + other * sn;
     }
     if (p.v_mix_mode == 1) {
       p.v_first[(size_t)t * p.v_first_stride + i] = x;
@@ -633,7 +641,7 @@ extern "C" int cpi_qkv_prepare(const void* qkv, int in_dtype, long qkv_stride, c
                                int interleaved, float* v_first, long v_first_stride, const void* v_mix,
                                int v_mix_dtype, int v_mix_mode, int maps, void* q2_out, void* k2_cache, int v_from_k,
                                int temperature, float floor_scale, float attn_scale, float rot_amp,
-                               cudaStream_t stream) {
+                               const float* v_inv_freq, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   CPI_REQUIRE(n_heads > 0 && n_kv_heads > 0 && n_heads % n_kv_heads == 0,
               "qkv_prepare: %d heads cannot be grouped over %d key/value heads", n_heads, n_kv_heads);
@@ -644,11 +652,13 @@ extern "C" int cpi_qkv_prepare(const void* qkv, int in_dtype, long qkv_stride, c
                   rot_dims, q_out, k_cache, v_cache, page_table, max_blocks, page_size, token_seq, token_pos,
                   seq_slot, n_heads, n_kv_heads, head_dim, v_dim, write_kv, head_norm, interleaved, v_first,
                   v_first_stride, v_mix, v_mix_dtype, v_mix_mode, maps, q2_out, k2_cache, v_from_k, temperature,
-                  floor_scale, attn_scale, rot_amp};
+                  floor_scale, attn_scale, rot_amp, v_inv_freq};
   CPI_REQUIRE(maps == 1 || (maps == 2 && q2_out != nullptr && (!write_kv || k2_cache != nullptr)),
               "qkv_prepare: one score map, or two with buffers for the second map's queries and keys");
   CPI_REQUIRE(!v_from_k || (maps == 1 && v_dim == head_dim && v_mix_mode == 0),
               "qkv_prepare: values that are the projected keys have the keys' size, one map and no value mixing");
+  CPI_REQUIRE(v_inv_freq == nullptr || (v_dim % 2 == 0 && v_mix_mode == 0),
+              "qkv_prepare: values that turn have an even size and are not mixed with other values");
   CPI_REQUIRE(!temperature || floor_scale > 0.f, "qkv_prepare: a query temperature needs a positive period");
   CPI_REQUIRE(!(head_norm && norm_whole), "qkv_prepare: a norm over the whole projection or one per head, not both");
   CPI_REQUIRE(head_norm >= 0 && head_norm <= 2, "qkv_prepare: unknown kind of head norm %d", head_norm);

@@ -1,7 +1,7 @@
 // Row-wise kernels: token embedding, RMS norm, row gather, expert-output combine.
 //
 // Formulas (file:line of kurulav1/cpi):
-//   embedding   x = Emb[token]                                   src/engine/llama4_cpu_engine.cpp:294-298
+//   embedding   x = Emb[token] * scale                            src/engine/llama4_cpu_engine.cpp:294-298
 //   rmsnorm     y = x * rsqrt(mean(x^2) + eps) * w, fp32 sums    src/engine/llama4_cpu_engine.cpp:47-62,
 //                                                                src/kernels/kernels.cu:36-99
 // The residual stream is float32 in both precisions; norm outputs take the activation dtype.
@@ -11,7 +11,7 @@ namespace cpi {
 
 template <typename TT>
 __global__ void embedding_kernel(const int* __restrict__ tokens, const TT* __restrict__ table,
-                                 float* __restrict__ out, int hidden, int vocab, int* __restrict__ err) {
+                                 float* __restrict__ out, int hidden, int vocab, float scale, int* __restrict__ err) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -30,12 +30,12 @@ __global__ void embedding_kernel(const int* __restrict__ tokens, const TT* __res
       const uint4 raw = r16[i];
       const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
       const float2 a = __bfloat1622float2(h2[0]), b = __bfloat1622float2(h2[1]), c = __bfloat1622float2(h2[2]), d = __bfloat1622float2(h2[3]);
-      reinterpret_cast<float4*>(dst)[2 * i] = make_float4(a.x, a.y, b.x, b.y);
-      reinterpret_cast<float4*>(dst)[2 * i + 1] = make_float4(c.x, c.y, d.x, d.y);
+      reinterpret_cast<float4*>(dst)[2 * i] = make_float4(a.x * scale, a.y * scale, b.x * scale, b.y * scale);
+      reinterpret_cast<float4*>(dst)[2 * i + 1] = make_float4(c.x * scale, c.y * scale, d.x * scale, d.y * scale);
     }
     return;
   }
-  for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = to_f32(row[i]);
+  for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = to_f32(row[i]) * scale;
 }
 
 // One block per row.  The sum of squares is taken in a fixed order (thread-strided, then a warp
@@ -412,11 +412,11 @@ extern "C" int cpi_gather_rows(const void* src, long src_stride_bytes, const int
 }
 
 extern "C" int cpi_embedding(const int* tokens, const void* table, int table_dtype, float* out,
-                             int n_tokens, int hidden, int vocab, int* err_flag, cudaStream_t stream) {
+                             int n_tokens, int hidden, int vocab, float scale, int* err_flag, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   CPI_REQUIRE(n_tokens > 0 && hidden > 0 && vocab > 0, "embedding: bad sizes T=%d H=%d V=%d", n_tokens, hidden, vocab);
   CPI_DISPATCH_DTYPE(table_dtype, TT,
-      cpi::launch_pdl(embedding_kernel<TT>, n_tokens, 256, 0, stream, tokens, (const TT*)table, out, hidden, vocab, err_flag));
+      cpi::launch_pdl(embedding_kernel<TT>, n_tokens, 256, 0, stream, tokens, (const TT*)table, out, hidden, vocab, scale, err_flag));
   return check_launch("embedding");
 }
 

@@ -7,7 +7,7 @@
 // [c | r] whose first part then goes through W_uv,h.  The two per-head products are grouped matrix products with one
 // group per head, over rows laid out head by head ("head-major": row h * T + t), which these kernels produce.
 //
-//   latent_kv_write     per token: c = rmsnorm(x[:rank]) * w, r = rotate(x[rank:rank + R]); the row [c | r] goes into
+//   latent_kv_write     per token: c = rmsnorm(x[:rank]) * w, r = rotate(x[rank:rank + R]) * amplitude; the row [c | r] goes into
 //                       the cache page of the token's position (one head of rank + R elements).
 //   latent_q_split      per token and head, from q [T, H, D + R] (float32): the first D elements go to the head-major
 //                       rows plain[h * T + t, :D]; the last R, rotated, to full[t, h, rank:rank + R].  Also fills the
@@ -30,6 +30,7 @@ struct LatentKvParams {
   const float* x; long x_stride;                 // [T, rank + R]
   const void* norm_w; int norm_dtype; float eps; // [rank] or null
   const float* inv_freq; int interleaved;        // [R / 2] or null
+  float amplitude;                               // of the rotation's sines and cosines
   void* cache;                                   // [pages, 1, page_size, rank + R]
   const int* page_table; int max_blocks; int page_size;
   const int* token_seq; const int* token_pos; const int* seq_slot;
@@ -66,6 +67,7 @@ __global__ void __launch_bounds__(256) latent_kv_write_kernel(LatentKvParams p) 
       const float other = x[p.rank + od];
       float sn, cs;
       sincosf((float)pos * p.inv_freq[f], &sn, &cs);
+      sn *= p.amplitude; cs *= p.amplitude;
       v = first ? v * cs - other * sn : v * cs + other * sn;
     }
     dst[p.rank + d] = from_f32<TO>(v);
@@ -74,7 +76,7 @@ __global__ void __launch_bounds__(256) latent_kv_write_kernel(LatentKvParams p) 
 
 struct LatentQParams {
   const float* q; long q_stride;                 // [T, H (D + R)]
-  const float* inv_freq; int interleaved;
+  const float* inv_freq; int interleaved; float amplitude;
   void* plain;                                   // [H T, D] head-major
   void* full;                                    // [T, H, rank + R]
   int* offsets; int* rows;                       // [H + 1], [H T]
@@ -106,6 +108,7 @@ __global__ void __launch_bounds__(256) latent_q_split_kernel(LatentQParams p) {
         const float other = q[i - r + od];
         float sn, cs;
         sincosf((float)pos * p.inv_freq[f], &sn, &cs);
+        sn *= p.amplitude; cs *= p.amplitude;
         v = first ? v * cs - other * sn : v * cs + other * sn;
       }
       full[(size_t)h * W + p.rank + r] = from_f32<TO>(v);
@@ -274,25 +277,25 @@ __global__ void __launch_bounds__(256) relu_squared_kernel(const float* x, long 
 using namespace cpi;
 
 extern "C" int cpi_latent_kv_write(const float* x, long x_stride, const void* norm_w, int norm_dtype, float eps,
-                                   const float* inv_freq, int interleaved, void* cache, int cache_dtype,
+                                   const float* inv_freq, int interleaved, float amplitude, void* cache, int cache_dtype,
                                    const int* page_table, int max_blocks, int page_size, const int* token_seq,
                                    const int* token_pos, const int* seq_slot, int n_tokens, int rank, int rot,
                                    cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   CPI_REQUIRE(rank >= 1 && rot >= 0 && rot % 2 == 0, "latent_kv_write: a latent of %d and a rotated part of %d", rank, rot);
-  LatentKvParams p{x, x_stride, norm_w, norm_dtype, eps, inv_freq, interleaved, cache, page_table, max_blocks,
+  LatentKvParams p{x, x_stride, norm_w, norm_dtype, eps, inv_freq, interleaved, amplitude, cache, page_table, max_blocks,
                    page_size, token_seq, token_pos, seq_slot, rank, rot};
   CPI_DISPATCH_DTYPE(cache_dtype, T, cpi::launch_pdl(latent_kv_write_kernel<T>, dim3(n_tokens), dim3(256), 0, stream, p));
   return check_launch("latent_kv_write");
 }
 
-extern "C" int cpi_latent_q_split(const float* q, long q_stride, const float* inv_freq, int interleaved, void* plain,
+extern "C" int cpi_latent_q_split(const float* q, long q_stride, const float* inv_freq, int interleaved, float amplitude, void* plain,
                                   void* full, int out_dtype, int* offsets, int* rows, const int* token_pos,
                                   int n_tokens, int n_heads, int dim, int rot, int rank, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   CPI_REQUIRE(n_heads >= 1 && dim >= 1 && rot >= 0 && rot % 2 == 0 && rank >= 1,
               "latent_q_split: bad sizes heads=%d dim=%d rotated=%d rank=%d", n_heads, dim, rot, rank);
-  LatentQParams p{q, q_stride, inv_freq, interleaved, plain, full, offsets, rows, token_pos, n_tokens, n_heads, dim,
+  LatentQParams p{q, q_stride, inv_freq, interleaved, amplitude, plain, full, offsets, rows, token_pos, n_tokens, n_heads, dim,
                   rot, rank};
   CPI_DISPATCH_DTYPE(out_dtype, T, cpi::launch_pdl(latent_q_split_kernel<T>, dim3(n_tokens), dim3(256), 0, stream, p));
   return check_launch("latent_q_split");

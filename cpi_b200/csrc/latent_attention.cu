@@ -15,7 +15,10 @@
 //                     (CH = 8 NT, NT = 8, 16 or 32 by the latent's size); V fragments through ldmatrix.trans
 //                     from the same shared-memory tile that held the keys
 // Key/value tiles are fetched with cp.async into two buffers, tile i + 1 while tile i is computed.  Rows of a tile
-// beyond the newest position are zero-filled, so stale page contents never reach a product.
+// beyond the newest position or before the block's first visible one are zero-filled, so stale page contents never reach a product.
+//
+// A window keeps a query to its own position and the ones just before it: tiles that no query of a block sees are
+// skipped, the rest is masked by position.
 //
 // Prefill: one block per group of consecutive tokens of a query tile (blockIdx.y) and per group of 64 heads.
 // Decode: one block per token, head group and key split; with more than one split the blocks leave unnormalised
@@ -41,6 +44,7 @@ struct Params {
   const float* sink;            // [H] or null
   int n_tokens, n_heads, row, rank;
   int heads_per_group, tokens_per_block, n_splits;
+  int window;                   // a query sees its own position and the window - 1 before it; 0: all before it
   float scale_log2;
 };
 
@@ -98,9 +102,11 @@ __global__ void __launch_bounds__(64 * RG, 1) latent_attention_kernel(Params p) 
 
   const int* table = p.page_table + (size_t)p.seq_slot[p.token_seq[tok0]] * p.max_blocks;
   const int last_pos = p.token_pos[tok0 + ntok - 1];
-  const int n_kv_tiles = last_pos / BN + 1;
+  // the first position that any query of the block sees (pages before it may have been given back and are not read)
+  const int first_pos = p.window > 0 ? max(0, p.token_pos[tok0] - p.window + 1) : 0;
+  const int first_tile = first_pos / BN, n_kv_tiles = last_pos / BN + 1 - first_tile;
   const int per_split = (n_kv_tiles + p.n_splits - 1) / p.n_splits;
-  const int t_begin = split * per_split, t_end = min(n_kv_tiles, t_begin + per_split);
+  const int t_begin = first_tile + split * per_split, t_end = min(first_tile + n_kv_tiles, t_begin + per_split);
   const int chunks = row >> 3;                                   // 16-byte pieces of a row
 
   // ---- queries: row m is token tok0 + m / HG, head hg0 + m % HG
@@ -121,7 +127,7 @@ __global__ void __launch_bounds__(64 * RG, 1) latent_attention_kernel(Params p) 
     for (int r = warp; r < BN; r += THREADS / 32) {
       const int kpos = tile * BN + r;
       __nv_bfloat16* dst = base + (size_t)r * LD;
-      if (kpos <= last_pos) {
+      if (kpos >= first_pos && kpos <= last_pos) {
         const int page = table[kpos / p.page_size];
         const __nv_bfloat16* src = p.cache + ((size_t)page * p.page_size + kpos % p.page_size) * row;
         for (int c = lane; c < chunks; c += 32) cp_async16(dst + c * 8, src + c * 8);
@@ -141,6 +147,8 @@ __global__ void __launch_bounds__(64 * RG, 1) latent_attention_kernel(Params p) 
   for (int i = 0; i < NT; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   const int col_base = ch * NT * 8;
+  const int reach = p.window > 0 ? p.window : 1 << 30;
+  auto sees = [&](int qp, int kp) { return kp <= qp && kp > qp - reach; };      // an empty row has qp = -1: no keys
 
   for (int it = t_begin; it < t_end; ++it) {
     const int buf = (it - t_begin) & 1;
@@ -179,10 +187,10 @@ __global__ void __launch_bounds__(64 * RG, 1) latent_attention_kernel(Params p) 
       for (int j = 0; j < 2; ++j) {
         const int col = ch * 16 + j * 8 + 2 * t4, kp = kv0 + col;
         float2 v0, v1;
-        v0.x = kp <= qp0 ? s[j][0] * p.scale_log2 : -INFINITY;
-        v0.y = kp + 1 <= qp0 ? s[j][1] * p.scale_log2 : -INFINITY;
-        v1.x = kp <= qp1 ? s[j][2] * p.scale_log2 : -INFINITY;
-        v1.y = kp + 1 <= qp1 ? s[j][3] * p.scale_log2 : -INFINITY;
+        v0.x = sees(qp0, kp) ? s[j][0] * p.scale_log2 : -INFINITY;
+        v0.y = sees(qp0, kp + 1) ? s[j][1] * p.scale_log2 : -INFINITY;
+        v1.x = sees(qp1, kp) ? s[j][2] * p.scale_log2 : -INFINITY;
+        v1.y = sees(qp1, kp + 1) ? s[j][3] * p.scale_log2 : -INFINITY;
         *reinterpret_cast<float2*>(Ss + r0 * SLD + col) = v0;
         *reinterpret_cast<float2*>(Ss + (r0 + 8) * SLD + col) = v1;
       }
@@ -373,7 +381,7 @@ extern "C" int cpi_latent_attention(const void* q, const void* cache, void* out,
                                     const int* token_pos, const int* seq_slot, const int* tile_tok0,
                                     const int* tile_rows, int n_tiles, int max_tile_rows, const float* sink,
                                     int n_tokens, int n_heads, int row, int rank, int n_splits, float scale,
-                                    cudaStream_t stream) {
+                                    int window, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   CPI_REQUIRE(cpi_latent_attention_supported(row, rank), "latent_attention: rows of %d with a latent of %d are not "
               "supported (multiples of 16, a latent of at most %d, a row of at most %d)", row, rank, lat::kMaxRank,
@@ -404,6 +412,7 @@ extern "C" int cpi_latent_attention(const void* q, const void* cache, void* out,
   p.heads_per_group = n_heads < bm ? n_heads : bm;
   p.tokens_per_block = bm / p.heads_per_group;
   p.n_splits = n_splits;
+  p.window = window > 0 ? window : 0;
   p.scale_log2 = scale * lat::kLog2e;
   const int head_groups = (n_heads + p.heads_per_group - 1) / p.heads_per_group;
   dim3 grid;

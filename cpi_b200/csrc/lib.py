@@ -24,7 +24,7 @@ MAX_DECODE_SPLITS = 256          # key splits that the combine kernel of decode 
 GENERAL_ATTENTION_MAX_DIM = 640  # largest key or value row of the general attention kernel
 PREFILL_TILE_ROWS = 256          # most query rows of one sequence that a block of the prefill attention kernel takes
 
-ABI_VERSION = 5                  # what cpi_abi_version() of a matching library answers
+ABI_VERSION = 6                  # what cpi_abi_version() of a matching library answers
 
 _lib = None
 scratch_generation = 0    # grows whenever a scratch buffer of this module is (re)allocated
@@ -93,14 +93,14 @@ def _rowmajor(t, what):
 
 
 # ------------------------------------------------------------------------------------------------
-def embedding(tokens, table, out, err_flag):
-    """out[t, :] = table[tokens[t], :] as float32; a token outside the table sets err_flag[0] = 1 + t."""
+def embedding(tokens, table, out, err_flag, scale=1.0):
+    """out[t, :] = table[tokens[t], :] * scale as float32; a token outside the table sets err_flag[0] = 1 + t."""
     _need_cuda(tokens, table, out, err_flag)
     T, H = out.shape
     assert tokens.dtype == torch.int32 and out.dtype == torch.float32 and out.is_contiguous()
     assert table.is_contiguous() and table.shape[1] == H
     _call("cpi_embedding", _p(tokens), _p(table), c_int(dtype_code(table.dtype)), _p(out), c_int(T), c_int(H),
-          c_int(table.shape[0]), _p(err_flag), _stream())
+          c_int(table.shape[0]), c_float(float(scale)), _p(err_flag), _stream())
 
 
 def rmsnorm(x, weight, eps, out, rows=None, weight_offset=0.0):
@@ -355,7 +355,7 @@ def qkv_prepare(qkv, q_out, k_cache, v_cache, page_table, page_size, token_seq, 
                 n_kv_heads, head_dim, value_dim, bias=None, q_norm=None, k_norm=None, norm_whole=False, norm_eps=0.0,
                 inv_freq=None, rotary_dims=0, write_kv=True, head_norm=False, interleaved=False, v_first=None,
                 v_mix=None, v_mix_mode=0, q2_out=None, k2_cache=None, values_from_keys=False, temperature=None,
-                rotary_amplitude=1.0):
+                rotary_amplitude=1.0, v_inv_freq=None):
     """The general form of `qkv_post`, a block per token: rows [q | k | v] (float32 or the cache's dtype) get
     their bias, q and k an RMS norm over the whole projection (`norm_whole`, weights `q_norm` / `k_norm`), the
     first `rotary_dims` elements of each head their rotation, and then (`head_norm` True or 1) every q and k head a
@@ -368,9 +368,11 @@ def qkv_prepare(qkv, q_out, k_cache, v_cache, page_table, page_size, token_seq, 
     k_cache, the second halves to q2_out and k2_cache (shaped alike); values have n_kv_heads heads.
     `values_from_keys`: rows are [q | k] and the cached values are the k rows as projected (bias added, before any
     norm).  `temperature` (f, a): q *= 1 + a * ln(floor((position + 1) / f) + 1).  `rotary_amplitude` multiplies the
-    rotation's sines and cosines."""
+    rotation's sines and cosines.  `v_inv_freq` (float32 [value_dim / 2]): the values turn too, over all their elements,
+    in the same layout of pairs."""
     _need_cuda(qkv, q_out, k_cache, v_cache, page_table, token_seq, token_pos, seq_slot, bias, q_norm, k_norm, inv_freq,
-               q2_out, k2_cache)
+               q2_out, k2_cache, v_inv_freq)
+    assert v_inv_freq is None or (v_inv_freq.dtype == torch.float32 and v_inv_freq.numel() == value_dim // 2)
     maps = 1 if q2_out is None else 2
     assert q2_out is None or (q2_out.is_contiguous() and q2_out.shape == q_out.shape and q2_out.dtype == q_out.dtype)
     assert k2_cache is None or (k2_cache.shape == k_cache.shape and k2_cache.dtype == k_cache.dtype)
@@ -397,7 +399,7 @@ def qkv_prepare(qkv, q_out, k_cache, v_cache, page_table, page_size, token_seq, 
           c_int(int(head_norm)), c_int(int(interleaved)), _p(v_first), c_long(0 if v_first is None else v_first.stride(0)),
           _p(v_mix), c_int(F32 if v_mix is None else dtype_code(v_mix.dtype)), c_int(int(v_mix_mode)), c_int(maps),
           _p(q2_out), _p(k2_cache), c_int(int(values_from_keys)), c_int(int(temperature is not None)), c_float(fl),
-          c_float(sc), c_float(float(rotary_amplitude)), _stream())
+          c_float(sc), c_float(float(rotary_amplitude)), _p(v_inv_freq), _stream())
 
 
 def head_post(a1, out, *, n_heads, value_dim, a2=None, lam=0.0, norm_eps=None, norm_scale=1.0, gate=None):
@@ -412,6 +414,91 @@ def head_post(a1, out, *, n_heads, value_dim, a2=None, lam=0.0, norm_eps=None, n
     _call("cpi_head_post", _p(a1), _p(a2), c_int(dtype_code(a1.dtype)), _p(out), c_int(dtype_code(out.dtype)),
           c_float(float(lam)), c_int(int(norm_eps is not None)), c_float(float(norm_eps or 0.0)), c_float(float(norm_scale)),
           _p(gate), c_long(0 if gate is None else gate.stride(0)), c_int(T), c_int(n_heads), c_int(value_dim), _stream())
+
+
+def qkv_conv_rotate_supported(head_dim, value_dim, rotary_dims, values_turn, taps) -> bool:
+    return bool(load().cpi_qkv_conv_rotate_supported(c_int(head_dim), c_int(value_dim), c_int(rotary_dims),
+                                                     c_int(int(values_turn)), c_int(taps)))
+
+
+def qkv_conv_rotate(qkv, q_out, k_cache, v_cache, page_table, page_size, batch, *, n_heads, n_kv_heads, head_dim, value_dim,
+                    conv_weight=None, carry=None, inv_freq=None, rotary_dims=0, v_inv_freq=None, interleaved=False,
+                    rotary_amplitude=1.0):
+    """From float32 rows [q | k | v] (a column slice of wider rows allowed): a causal convolution over time per channel
+    (`conv_weight` float32 [taps, channels]: TRANSPOSED against `causal_conv`; inputs before the step from `carry`
+    [slots, taps - 1, channels], which afterwards holds each sequence's last inputs), the rotation of q and k over their
+    first `rotary_dims` elements, the rotation of v over all of its elements (`v_inv_freq`); q to q_out, k and v into the
+    cache pages.  For the sizes that `qkv_conv_rotate_supported` takes; others go through `causal_conv` and
+    `qkv_prepare`."""
+    _need_cuda(qkv, q_out, k_cache, v_cache, page_table, conv_weight, carry, inv_freq, v_inv_freq)
+    T, C = qkv.shape
+    assert C == n_heads * head_dim + n_kv_heads * (head_dim + value_dim) and qkv.dtype == torch.float32 and qkv.stride(1) == 1
+    assert q_out.is_contiguous() and q_out.shape == (T, n_heads * head_dim) and k_cache.dtype == v_cache.dtype == q_out.dtype
+    assert k_cache.is_contiguous() and v_cache.is_contiguous()
+    assert k_cache.shape[-1] == head_dim and v_cache.shape[-1] == value_dim
+    assert inv_freq is None or (inv_freq.dtype == torch.float32 and inv_freq.numel() == rotary_dims // 2)
+    assert v_inv_freq is None or (v_inv_freq.dtype == torch.float32 and v_inv_freq.numel() == value_dim // 2)
+    taps = 1 if conv_weight is None else conv_weight.shape[0]
+    if conv_weight is not None:
+        assert conv_weight.dtype == torch.float32 and conv_weight.is_contiguous() and conv_weight.shape[1] == C
+        assert carry.dtype == torch.float32 and carry.is_contiguous() and tuple(carry.shape[1:]) == (taps - 1, C)
+    tiles = None if batch.is_decode else (batch.tile_tok0, batch.tile_rows)
+    _call("cpi_qkv_conv_rotate", _p(qkv), c_long(qkv.stride(0)), _p(conv_weight), c_int(taps), _p(carry), _p(inv_freq),
+          c_int(rotary_dims), _p(v_inv_freq), c_int(int(interleaved)), c_float(float(rotary_amplitude)), _p(q_out),
+          _p(k_cache), _p(v_cache), c_int(dtype_code(q_out.dtype)), _p(page_table), c_int(page_table.shape[1]),
+          c_int(page_size), _p(batch.token_seq), _p(batch.token_pos), _p(batch.seq_slot), _p(batch.seq_start),
+          _p(tiles[0] if tiles else None), _p(tiles[1] if tiles else None), c_int(batch.n_q_tiles if tiles else 0),
+          c_int(PREFILL_TILE_ROWS), c_int(T), c_int(n_heads), c_int(n_kv_heads), c_int(head_dim), c_int(value_dim), _stream())
+    if tiles and taps > 1:              # a step of single tokens has updated the carried inputs itself
+        _call("cpi_conv_carry_rows", _p(qkv), c_long(qkv.stride(0)), _p(carry), c_int(C), c_int(taps), _p(batch.seq_slot),
+              _p(batch.seq_tok0), _p(batch.seq_new), c_int(batch.n_seqs), _stream())
+
+
+def head_turn(x, out, token_pos, *, n_heads, value_dim, inv_freq=None, interleaved=False, gate=None):
+    """Per token and head: the head's output x [T, heads * value_dim] turned back by the token's position (`inv_freq`
+    float32 [value_dim / 2], None: not turned), times sigmoid(gate) element by element (`gate` float32 [T, heads *
+    value_dim], a column slice allowed; None: no gate); rounded once into out, which may be x."""
+    _need_cuda(x, out, token_pos, gate, inv_freq)
+    T, W = x.shape
+    assert W == n_heads * value_dim and x.is_contiguous() and out.is_contiguous() and out.shape == x.shape and out.dtype == x.dtype
+    assert inv_freq is None or (inv_freq.dtype == torch.float32 and inv_freq.numel() == value_dim // 2)
+    assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape == (T, W))
+    _call("cpi_head_turn", _p(x), _p(out), c_int(dtype_code(x.dtype)), _p(gate), c_long(0 if gate is None else gate.stride(0)),
+          _p(inv_freq), c_int(int(interleaved)), _p(token_pos), c_int(T), c_int(n_heads), c_int(value_dim), _stream())
+
+
+def norm_step(x, *, y=None, experts=None, post=None, pre=None, h_out=None, rows=None, add=True):
+    """One boundary between sublayers whose norms are n(v) = tanh(alpha v) * w + b (`post`, `pre`: (alpha, w, b) with
+    float32 [W] vectors).  x (float32 [T, W], in place) (+)= post(v), v being the row y[t] (float32) or the sum over a
+    token's chosen experts; then h_out = pre(x), of the rows `rows` names if given.  `experts`: (ye float32 [*, W] weighted
+    output rows, row_of_slot int32 [T, k], expert int32 [T, k], weight float32 [T, k], h [T, W], number of experts that
+    have rows): a chosen expert beyond that number contributes weight * h[t].  post None: v as it is.  add False: x is
+    replaced."""
+    _need_cuda(x, y, h_out, rows)
+    T, W = x.shape
+    assert x.dtype == torch.float32 and x.stride(1) == 1
+    assert y is None or (y.dtype == torch.float32 and y.shape == (T, W) and y.stride(1) == 1)
+    ye = ros = idx = wt = h = None
+    top_k = n_real = 0
+    if experts is not None:
+        ye, ros, idx, wt, h, n_real = experts
+        _need_cuda(ye, ros, idx, wt, h)
+        top_k = idx.shape[-1]
+        assert ye.dtype == torch.float32 and ye.is_contiguous() and ye.shape[-1] == W and h.shape == (T, W) and h.stride(1) == 1
+        assert ros.dtype == idx.dtype == torch.int32 and wt.dtype == torch.float32
+        assert ros.numel() == idx.numel() == wt.numel() == T * top_k and ros.is_contiguous() and idx.is_contiguous()
+    n = T if rows is None else rows.numel()
+    assert h_out is None or (h_out.shape == (n, W) and h_out.stride(1) == 1)
+    assert rows is None or rows.dtype == torch.int32
+    for norm in (post, pre):
+        assert norm is None or all(t.is_cuda and t.dtype == torch.float32 and t.is_contiguous() and t.numel() == W for t in norm[1:])
+    a, b = post or (0.0, None, None), pre or (0.0, None, None)
+    _call("cpi_norm_step", _p(y), c_long(0 if y is None else y.stride(0)), _p(ye), _p(ros), _p(idx), _p(wt), _p(h),
+          c_int(F32 if h is None else dtype_code(h.dtype)), c_long(0 if h is None else h.stride(0)), c_int(top_k),
+          c_int(n_real), _p(x), c_long(x.stride(0)), c_int(int(add)), c_int(int(post is not None)), c_float(a[0]), _p(a[1]),
+          _p(a[2]), c_int(int(pre is not None)), c_float(b[0]), _p(b[1]), _p(b[2]), _p(h_out),
+          c_int(F32 if h_out is None else dtype_code(h_out.dtype)), c_long(0 if h_out is None else h_out.stride(0)), _p(rows),
+          c_int(n), c_int(W), _stream())
 
 
 def sum_norm_add(branches, scales, weight, out, *, eps=0.0, add=True, h_out=None, normalise=True):
@@ -479,9 +566,9 @@ def rglru_scan(gates, u, y, state, out, batch, *, block, lam, r_bias=None, i_bia
 
 
 def latent_kv_write(x, norm_weight, eps, inv_freq, interleaved, cache, page_table, page_size, token_seq, token_pos,
-                    seq_slot, *, rank, rot):
+                    seq_slot, *, rank, rot, amplitude=1.0):
     """Per token, from float32 rows x [T, rank + rot] (a column slice allowed): the first `rank` elements RMS-normed
-    (times `norm_weight`), the last `rot` rotated by the token's position; the row goes into the page of its position
+    (times `norm_weight`), the last `rot` rotated by the token's position (sines and cosines times `amplitude`); the row goes into the page of its position
     in `cache` [pages, 1, page_size, rank + rot]."""
     _need_cuda(x, norm_weight, inv_freq, cache, page_table, token_seq, token_pos, seq_slot)
     assert x.dtype == torch.float32 and x.dim() == 2 and x.stride(1) == 1 and x.shape[1] == rank + rot
@@ -490,12 +577,13 @@ def latent_kv_write(x, norm_weight, eps, inv_freq, interleaved, cache, page_tabl
     assert norm_weight is None or (norm_weight.is_contiguous() and norm_weight.numel() == rank)
     _call("cpi_latent_kv_write", _p(x), c_long(x.stride(0)), _p(norm_weight),
           c_int(F32 if norm_weight is None else dtype_code(norm_weight.dtype)), c_float(eps), _p(inv_freq),
-          c_int(int(interleaved)), _p(cache), c_int(dtype_code(cache.dtype)), _p(page_table), c_int(page_table.shape[1]),
+          c_int(int(interleaved)), c_float(float(amplitude)), _p(cache), c_int(dtype_code(cache.dtype)), _p(page_table), c_int(page_table.shape[1]),
           c_int(page_size), _p(token_seq), _p(token_pos), _p(seq_slot), c_int(x.shape[0]), c_int(rank), c_int(rot),
           _stream())
 
 
-def latent_q_split(q, inv_freq, interleaved, plain, full, offsets, rows, token_pos, *, n_heads, dim, rot, rank):
+def latent_q_split(q, inv_freq, interleaved, plain, full, offsets, rows, token_pos, *, n_heads, dim, rot, rank,
+                   amplitude=1.0):
     """From float32 rows q [T, heads * (dim + rot)]: a head's first `dim` elements go to plain[head * T + t] (rows laid
     out head by head), its last `rot`, rotated by the token's position, to full[t, head, rank : rank + rot].  Also
     fills offsets[h] = h * T (int32 [heads + 1]) and rows[h * T + t] = t * heads + h (int32 [heads * T])."""
@@ -506,7 +594,8 @@ def latent_q_split(q, inv_freq, interleaved, plain, full, offsets, rows, token_p
     assert full.is_contiguous() and full.numel() == T * n_heads * (rank + rot)
     assert offsets.dtype == torch.int32 and offsets.numel() >= n_heads + 1 and rows.dtype == torch.int32
     assert rows.numel() >= T * n_heads
-    _call("cpi_latent_q_split", _p(q), c_long(q.stride(0)), _p(inv_freq), c_int(int(interleaved)), _p(plain), _p(full),
+    _call("cpi_latent_q_split", _p(q), c_long(q.stride(0)), _p(inv_freq), c_int(int(interleaved)), c_float(float(amplitude)),
+          _p(plain), _p(full),
           c_int(dtype_code(full.dtype)), _p(offsets), _p(rows), _p(token_pos), c_int(T), c_int(n_heads), c_int(dim),
           c_int(rot), c_int(rank), _stream())
 
@@ -771,12 +860,13 @@ LATENT_KEY_TILE = 32             # cached positions that a block of the latent a
 
 
 def latent_attention(q, out, cache, page_table, page_size, token_seq, token_pos, seq_slot, *, n_heads, rank, scale,
-                     sink=None, tile_tok0=None, tile_rows=None, n_splits=1):
+                     sink=None, tile_tok0=None, tile_rows=None, n_splits=1, window=0):
     """bfloat16 softmax attention of q [T, heads * row] over cached rows [pages, 1, page_size, row] that all heads
     share: a row is the key, its first `rank` elements the value; a query sees every position up to its own.  out
     [heads * T, rank] is laid out head by head (row h * T + t).  With `tile_tok0` / `tile_rows` (runs of at most
     PREFILL_TILE_ROWS consecutive tokens of one sequence) a block takes a few tokens of a run; without, every token
-    is alone and its keys are divided over `n_splits` blocks.  `sink`: float32 [heads], joins the denominators."""
+    is alone and its keys are divided over `n_splits` blocks.  `sink`: float32 [heads], joins the denominators.
+    `window` n > 0: a query sees its own position and the n - 1 before it."""
     _need_cuda(q, out, cache, page_table, token_seq, token_pos, seq_slot, sink, tile_tok0, tile_rows)
     T = q.shape[0]
     row = cache.shape[-1]
@@ -799,7 +889,7 @@ def latent_attention(q, out, cache, page_table, page_size, token_seq, token_pos,
     _call("cpi_latent_attention", _p(q), _p(cache), _p(out), _p(po), _p(pml), _p(page_table),
           c_int(page_table.shape[1]), c_int(page_size), _p(token_seq), _p(token_pos), _p(seq_slot), _p(tile_tok0),
           _p(tile_rows), c_int(0 if tile_tok0 is None else tile_tok0.numel()), c_int(PREFILL_TILE_ROWS), _p(sink),
-          c_int(T), c_int(n_heads), c_int(row), c_int(rank), c_int(int(n_splits)), c_float(scale), _stream())
+          c_int(T), c_int(n_heads), c_int(row), c_int(rank), c_int(int(n_splits)), c_float(scale), c_int(int(window)), _stream())
 
 
 def attention_decode_blocks_per_sm(head_dim: int) -> int:
@@ -828,18 +918,22 @@ def attention_prefill(q, out, k_cache, v_cache, page_table, page_size, token_seq
           _p(sink), c_int(int(keep_first)), c_float(float(softcap or 0.0)), _stream())
 
 
-ROUTER_GATES = {"none": 0, "sigmoid": 1, "softmax_chosen": 2, "sigmoid_normed": 3}
+ROUTER_GATES = {"none": 0, "sigmoid": 1, "softmax_chosen": 2, "sigmoid_normed": 3, "scored": 3}
 
 
 def _rule(rule):
-    """The extra arguments of the selection: `rule` None, or for the gate "sigmoid_normed" a dictionary {"choice_bias":
-    float32 [experts] or None, "groups": n, "keep": n, "scale": s}: the choice is made on sigmoid(logit) + choice_bias
-    among the experts of the `keep` best of `groups` equal groups (a group's score: its two largest choice scores
-    summed), the weights are the chosen sigmoids divided by their sum and multiplied by `scale`."""
+    """The extra arguments of the selection by scores (the gates "sigmoid_normed" and "scored"): a dictionary {"score":
+    "sigmoid" | "softmax" (over all of a token's logits), "choice_bias": float32 [experts] or None, "groups": n, "keep": n,
+    "group_score": "top2_sum" | "max", "normalise": bool, "scale": s}: the choice is made on score + choice_bias among the
+    experts of the `keep` best of `groups` equal groups (a group's score: its two largest choice scores summed, or the
+    largest), the weights are the chosen scores, divided by their sum if `normalise`, times `scale`."""
     r = rule or {}
     cb = r.get("choice_bias")
     assert cb is None or (cb.dtype == torch.float32 and cb.is_contiguous() and cb.is_cuda)
-    return _p(cb), c_int(int(r.get("groups", 1))), c_int(int(r.get("keep", 1))), c_float(float(r.get("scale", 1.0)))
+    flavour = (int(r.get("score", "sigmoid") == "softmax") | 2 * int(r.get("group_score", "top2_sum") == "max")
+               | 4 * int(not r.get("normalise", True)))
+    return (_p(cb), c_int(int(r.get("groups", 1))), c_int(int(r.get("keep", 1))), c_float(float(r.get("scale", 1.0))),
+            c_int(flavour))
 
 
 def _gate_mode(sigmoid_gate) -> int:

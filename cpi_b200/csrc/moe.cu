@@ -136,77 +136,131 @@ router_logits_tile_kernel(const TH* __restrict__ h, long h_stride, const TW* __r
   }
 }
 
-// Mode 3 of the selection: scores s = sigmoid(logit); the choice is made on s + choice_bias (the bias never enters a
-// weight); the experts form `n_groups` equal groups of neighbours, a group's score is the sum of its two largest choice
-// scores, and only experts of the `keep_groups` best groups can be chosen; the weights are the chosen s divided by their
-// sum (+ 1e-20), times `gate_scale`.
+// Mode 3 of the selection: scores s = sigmoid(logit), or (flavour bit 0) the softmax over all of a token's logits; the
+// choice is made on s + choice_bias (the bias never enters a weight); the experts form `n_groups` equal groups of
+// neighbours, a group's score is the sum of its two largest choice scores, or (bit 1) its largest, and only experts of
+// the `keep_groups` best groups can be chosen (the others are left out, not zeroed: choice scores may be negative); the
+// weights are the chosen s divided by their sum (+ 1e-20), or (bit 2) as they are, times `gate_scale`.
+enum SelectFlavour : int { kScoreSoftmax = 1, kGroupLargest = 2, kWeightsAsScored = 4 };
 struct SelectRule {
   int gate_mode;
   const float* choice_bias;              // [experts] float32 or null
   int n_groups, keep_groups;             // 1, 1: no groups
   float gate_scale;
+  int flavour;
 };
 
-__device__ __forceinline__ void select_grouped(const float* lg, int* idx, float* gate, int n_experts, int top_k,
-                                               const SelectRule& r) {
-  auto choice = [&](int e) {
-    const float s = 1.0f / (1.0f + expf(-lg[e]));
-    return r.choice_bias ? s + r.choice_bias[e] : s;
-  };
-  const int per = n_experts / r.n_groups;
-  unsigned long long kept = ~0ull;
-  if (r.n_groups > 1 && r.keep_groups < r.n_groups) {
-    kept = 0ull;
-    for (int k = 0; k < r.keep_groups; ++k) {
-      int bg = -1;
-      float bs = 0.f;
-      for (int g = 0; g < r.n_groups; ++g) {
-        if ((kept >> g) & 1ull) continue;
-        float m1 = -INFINITY, m2 = -INFINITY;              // the group's two largest choice scores
-        for (int e = g * per; e < (g + 1) * per; ++e) {
-          const float c = choice(e);
-          if (c != c) continue;
-          if (c > m1) { m2 = m1; m1 = c; } else if (c > m2) { m2 = c; }
-        }
-        const float gs = per > 1 ? m1 + m2 : m1;
-        if (bg < 0 || gs > bs) { bg = g; bs = gs; }
-      }
-      kept |= 1ull << bg;
+// One warp per token; lane l holds experts l, l + 32, ...  Every comparison takes the lower index at a tie and never a
+// NaN, and every sum has one order, so a token's choice depends on its logits alone.
+__device__ __forceinline__ void warp_best(float& v, int& i) {      // the largest v, ties to the lowest i; i < 0: nothing
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, i, o);
+    if (oi >= 0 && (i < 0 || ov > v || (ov == v && oi < i))) { v = ov; i = oi; }
+  }
+}
+
+__device__ __forceinline__ void select_scored_warp(const float* lg, int* idx, float* gate, int n_experts, int top_k,
+                                                   const SelectRule& r) {
+  constexpr int PER = kMaxExperts / 32;
+  const int lane = threadIdx.x & 31;
+  float s[PER], c[PER];
+  if (r.flavour & kScoreSoftmax) {
+    float mx = -INFINITY, sum = 0.f;
+#pragma unroll
+    for (int j = 0; j < PER; ++j) {
+      const int e = lane + 32 * j;
+      s[j] = e < n_experts ? lg[e] : -INFINITY;
+      mx = fmaxf(mx, s[j]);
     }
+    mx = warp_max(mx);
+#pragma unroll
+    for (int j = 0; j < PER; ++j) { s[j] = lane + 32 * j < n_experts ? expf(s[j] - mx) : 0.f; sum += s[j]; }
+    sum = warp_sum(sum);
+#pragma unroll
+    for (int j = 0; j < PER; ++j) s[j] /= sum;
+  } else {
+#pragma unroll
+    for (int j = 0; j < PER; ++j) { const int e = lane + 32 * j; s[j] = e < n_experts ? 1.0f / (1.0f + expf(-lg[e])) : 0.f; }
+  }
+#pragma unroll
+  for (int j = 0; j < PER; ++j) {
+    const int e = lane + 32 * j;
+    c[j] = e < n_experts && r.choice_bias ? s[j] + r.choice_bias[e] : s[j];
+  }
+  unsigned open = 0;                     // bit j: expert lane + 32 j can (still) be chosen
+  const int per = n_experts / r.n_groups;
+#pragma unroll
+  for (int j = 0; j < PER; ++j) open |= (lane + 32 * j < n_experts && c[j] == c[j]) ? 1u << j : 0u;
+  if (r.n_groups > 1 && r.keep_groups < r.n_groups) {
+    // lane g and lane g + 32 hold the scores of groups g and g + 32 (up to 64)
+    float gs[2] = {-INFINITY, -INFINITY};
+    for (int g = 0; g < r.n_groups; ++g) {
+      float total = 0.f;
+      int first = -1;
+      for (int pass = 0; pass < ((r.flavour & kGroupLargest) || per < 2 ? 1 : 2); ++pass) {
+        float v = -INFINITY;
+        int i = -1;
+#pragma unroll
+        for (int j = 0; j < PER; ++j) {
+          const int e = lane + 32 * j;
+          if (((open >> j) & 1u) && e / per == g && e != first && (i < 0 || c[j] > v)) { v = c[j]; i = e; }
+        }
+        warp_best(v, i);
+        total = pass == 0 ? v : total + v;
+        first = i;
+      }
+      if ((g & 31) == lane) gs[g >> 5] = total;
+    }
+    unsigned long long kept = 0ull;
+    for (int k = 0; k < r.keep_groups; ++k) {
+      float v = 0.f;
+      int i = -1;
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const int g = lane + 32 * u;
+        if (g < r.n_groups && !((kept >> g) & 1ull) && (i < 0 || gs[u] > v)) { v = gs[u]; i = g; }
+      }
+      warp_best(v, i);
+      kept |= 1ull << i;
+    }
+#pragma unroll
+    for (int j = 0; j < PER; ++j)
+      if (lane + 32 * j < n_experts && !((kept >> ((lane + 32 * j) / per)) & 1ull)) open &= ~(1u << j);
   }
   float sum = 0.f;
+  unsigned taken = 0;
   for (int k = 0; k < top_k; ++k) {
-    int best = -1;
-    float bv = 0.f;
-    for (int e = 0; e < n_experts; ++e) {
-      if (!((kept >> (e / per)) & 1ull)) continue;
-      bool taken = false;
-      for (int j = 0; j < k; ++j) taken |= (idx[j] == e);
-      if (taken) continue;
-      const float c = choice(e);
-      if (c != c) continue;
-      if (best < 0 || c > bv) { best = e; bv = c; }
+    float v = 0.f, sc = 0.f;
+    int i = -1;
+#pragma unroll
+    for (int j = 0; j < PER; ++j)
+      if (((open >> j) & 1u) && (i < 0 || c[j] > v)) { v = c[j]; i = lane + 32 * j; }
+    warp_best(v, i);
+    if (i < 0) {                         // nothing left to choose from: the lowest free index
+      int f = n_experts;
+#pragma unroll
+      for (int j = PER - 1; j >= 0; --j)
+        if (lane + 32 * j < n_experts && !((taken >> j) & 1u)) f = lane + 32 * j;
+      i = -__reduce_max_sync(0xffffffffu, -f);
     }
-    if (best < 0) {                                        // nothing left to choose from: the lowest free index
-      for (int e = 0; e < n_experts && best < 0; ++e) {
-        bool taken = false;
-        for (int j = 0; j < k; ++j) taken |= (idx[j] == e);
-        if (!taken) best = e;
-      }
-    }
-    idx[k] = best;
-    gate[k] = 1.0f / (1.0f + expf(-lg[best]));
-    sum += gate[k];
+#pragma unroll
+    for (int j = 0; j < PER; ++j)
+      if (lane + 32 * j == i) { open &= ~(1u << j); taken |= 1u << j; sc = s[j]; }
+    sc = __shfl_sync(0xffffffffu, sc, i & 31);
+    if (lane == 0) { idx[k] = i; gate[k] = sc; }
+    sum += sc;
   }
-  const float f = r.gate_scale / (sum + 1e-20f);
-  for (int k = 0; k < top_k; ++k) gate[k] *= f;
+  const float f = r.flavour & kWeightsAsScored ? r.gate_scale : r.gate_scale / (sum + 1e-20f);
+  if (lane == 0)
+    for (int k = 0; k < top_k; ++k) gate[k] *= f;
 }
 
 // The k best logits of one token, ties to the lowest index; gate = 1 (mode 0), the sigmoid of the chosen logit
-// (mode 1), or the softmax over the chosen logits (mode 2); mode 3: see SelectRule.
+// (mode 1), or the softmax over the chosen logits (mode 2).
 __device__ __forceinline__ void select_topk(const float* lg, int* idx, float* gate, int n_experts, int top_k, const SelectRule& rule) {
   const int gate_mode = rule.gate_mode;
-  if (gate_mode == 3) { select_grouped(lg, idx, gate, n_experts, top_k, rule); return; }
   for (int k = 0; k < top_k; ++k) {
     int best = -1;
     float bv = 0.f;
@@ -236,6 +290,18 @@ __device__ __forceinline__ void select_topk(const float* lg, int* idx, float* ga
     const float inv = 1.0f / sum;
     for (int k = 0; k < top_k; ++k) gate[k] *= inv;
   }
+}
+
+// Mode 3: a warp per token.
+__global__ void __launch_bounds__(128) router_select_scored_kernel(const float* __restrict__ logits, int* __restrict__ topk_idx,
+                                                                   float* __restrict__ topk_gate, int n_tokens, int n_experts,
+                                                                   int top_k, SelectRule rule) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (t >= n_tokens) return;
+  select_scored_warp(logits + (size_t)t * n_experts, topk_idx + (size_t)t * top_k, topk_gate + (size_t)t * top_k, n_experts,
+                     top_k, rule);
 }
 
 // One thread per token.
@@ -268,8 +334,13 @@ moe_route_small_kernel(const float* __restrict__ logits, int n_tokens, int n_exp
   const int tid = threadIdx.x, M = n_tokens * top_k;
   for (int i = tid; i < n_tokens * n_experts; i += 128) lg_s[i] = logits[i];
   __syncthreads();
-  for (int t = tid; t < n_tokens; t += 128)
-    select_topk(lg_s + t * n_experts, idx_s + t * top_k, gate_s + t * top_k, n_experts, top_k, rule);
+  if (rule.gate_mode == 3) {
+    for (int t = tid >> 5; t < n_tokens; t += 4)
+      select_scored_warp(lg_s + t * n_experts, idx_s + t * top_k, gate_s + t * top_k, n_experts, top_k, rule);
+  } else {
+    for (int t = tid; t < n_tokens; t += 128)
+      select_topk(lg_s + t * n_experts, idx_s + t * top_k, gate_s + t * top_k, n_experts, top_k, rule);
+  }
   __syncthreads();
   for (int e = tid; e < n_experts; e += 128) {
     int c = 0;
@@ -371,6 +442,15 @@ moe_lists_kernel(const int* __restrict__ topk_idx, const float* __restrict__ top
 
 using namespace cpi;
 
+static int launch_select(const float* logits, int* topk_idx, float* topk_gate, int n_tokens, int n_experts, int top_k,
+                         const SelectRule& rule, cudaStream_t stream) {
+  if (rule.gate_mode == 3)
+    cpi::launch_pdl(router_select_scored_kernel, (n_tokens + 3) / 4, 128, 0, stream, logits, topk_idx, topk_gate, n_tokens, n_experts, top_k, rule);
+  else
+    cpi::launch_pdl(router_select_kernel, (n_tokens + 127) / 128, 128, 0, stream, logits, topk_idx, topk_gate, n_tokens, n_experts, top_k, rule);
+  return check_launch("router_select");
+}
+
 static int check_rule(const SelectRule& r, int n_experts) {
   if (r.gate_mode != 3) return 0;
   CPI_REQUIRE(r.n_groups >= 1 && r.n_groups <= 64 && n_experts % r.n_groups == 0 && r.keep_groups >= 1 &&
@@ -387,7 +467,7 @@ extern "C" int cpi_router_topk(const void* h, int h_dtype, long h_stride, const 
                                float* logits, int* topk_idx, float* topk_gate, int n_tokens,
                                int hidden, int n_experts, int top_k, int gate_mode, const float* bias,
                                int sigmoid_out, const float* choice_bias, int n_groups, int keep_groups,
-                               float gate_scale, cudaStream_t stream) {
+                               float gate_scale, int flavour, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
   CPI_REQUIRE(n_experts >= 1 && n_experts <= kMaxExperts, "router: %d experts (supported: 1..%d)", n_experts, kMaxExperts);
   CPI_REQUIRE(top_k >= 1 && top_k <= n_experts, "router: top-k %d of %d experts", top_k, n_experts);
@@ -409,10 +489,9 @@ extern "C" int cpi_router_topk(const void* h, int h_dtype, long h_stride, const 
   }
   if (check_launch("router_logits")) return 2;
   if (!topk_idx) return 0;                          // logits only: the caller selects in a later kernel
-  SelectRule rule{gate_mode, choice_bias, n_groups, keep_groups, gate_scale};
+  SelectRule rule{gate_mode, choice_bias, n_groups, keep_groups, gate_scale, flavour};
   if (check_rule(rule, n_experts)) return 1;
-  cpi::launch_pdl(router_select_kernel, (n_tokens + 127) / 128, 128, 0, stream, logits, topk_idx, topk_gate, n_tokens, n_experts, top_k, rule);
-  return check_launch("router_select");
+  return launch_select(logits, topk_idx, topk_gate, n_tokens, n_experts, top_k, rule, stream);
 }
 
 // Selection, lists and (when sorted_h is given) the gather for logits already computed: one launch for a
@@ -421,14 +500,14 @@ extern "C" int cpi_moe_route_small(const float* logits, int n_tokens, int n_expe
                                    int* topk_idx, float* topk_gate, int* group_offsets, int* row_token,
                                    float* row_scale, int* row_of_slot, const void* h, long h_stride_bytes,
                                    void* sorted_h, int row_bytes, const float* choice_bias, int n_groups,
-                                   int keep_groups, float gate_scale, cudaStream_t stream) {
+                                   int keep_groups, float gate_scale, int flavour, cudaStream_t stream) {
   if (n_tokens <= 0 || (long)n_tokens * top_k > kSmallSlots || (long)n_tokens * n_experts > kSmallLogits ||
       n_experts > kMaxExperts || top_k < 1 || top_k > n_experts)
     return -1;
   if (sorted_h && (row_bytes % 16 || h_stride_bytes % 16 || (reinterpret_cast<uintptr_t>(h) & 15) ||
                    (reinterpret_cast<uintptr_t>(sorted_h) & 15)))
     return -1;
-  SelectRule rule{gate_mode, choice_bias, n_groups, keep_groups, gate_scale};
+  SelectRule rule{gate_mode, choice_bias, n_groups, keep_groups, gate_scale, flavour};
   if (check_rule(rule, n_experts)) return 1;
   cpi::launch_pdl(moe_route_small_kernel, n_tokens * top_k, 128, 0, stream, logits, n_tokens, n_experts, top_k, rule,
                   topk_idx, topk_gate, group_offsets, row_token, row_scale, row_of_slot,
@@ -438,12 +517,11 @@ extern "C" int cpi_moe_route_small(const float* logits, int n_tokens, int n_expe
 
 extern "C" int cpi_router_select(const float* logits, int* topk_idx, float* topk_gate, int n_tokens, int n_experts,
                                  int top_k, int gate_mode, const float* choice_bias, int n_groups, int keep_groups,
-                                 float gate_scale, cudaStream_t stream) {
+                                 float gate_scale, int flavour, cudaStream_t stream) {
   if (n_tokens == 0) return 0;
-  SelectRule rule{gate_mode, choice_bias, n_groups, keep_groups, gate_scale};
+  SelectRule rule{gate_mode, choice_bias, n_groups, keep_groups, gate_scale, flavour};
   if (check_rule(rule, n_experts)) return 1;
-  cpi::launch_pdl(router_select_kernel, (n_tokens + 127) / 128, 128, 0, stream, logits, topk_idx, topk_gate, n_tokens, n_experts, top_k, rule);
-  return check_launch("router_select");
+  return launch_select(logits, topk_idx, topk_gate, n_tokens, n_experts, top_k, rule, stream);
 }
 
 extern "C" int cpi_moe_lists(const int* topk_idx, const float* topk_gate, int* group_offsets, int* row_token,

@@ -21,10 +21,12 @@ class Layer:
     feed_forward: object
     mixer_norm: object
     feed_forward_norm: object
+    mixer_post_norm: object = None
+    feed_forward_post_norm: object = None
 
     def parts(self):
-        return tuple(p for p in (self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward)
-                     if p is not None)
+        return tuple(p for p in (self.mixer_norm, self.mixer, self.mixer_post_norm, self.feed_forward_norm,
+                                 self.feed_forward, self.feed_forward_post_norm) if p is not None)
 
     def all_parts(self):
         """Every object whose code runs in a step of this layer (the mixer's position encoding included)."""
@@ -56,6 +58,10 @@ class DecoderModel:
                 mixer_norm=build_part("norm", ls.mixer_norm, ls.prefix, workspace=self.ws, tag="norm_mixer"),
                 feed_forward_norm=None if ls.feed_forward is None or ls.feed_forward_norm is None else
                 build_part("norm", ls.feed_forward_norm, ls.prefix, workspace=self.ws, tag="norm_ffn"),
+                mixer_post_norm=None if ls.mixer_post_norm is None else
+                build_part("norm", ls.mixer_post_norm, ls.prefix, workspace=self.ws, tag="norm_mixer_out"),
+                feed_forward_post_norm=None if ls.feed_forward is None or ls.feed_forward_post_norm is None else
+                build_part("norm", ls.feed_forward_post_norm, ls.prefix, workspace=self.ws, tag="norm_ffn_out"),
             ))
         self.streams = int(spec.residual_streams)
         if self.streams < 1:
@@ -71,6 +77,7 @@ class DecoderModel:
         if self.embed_norm is not None and self.streams != 1:
             raise ValueError("a norm on the embedding output does not combine with several residual streams")
         self.embed_name = spec.embedding["weight"]
+        self.embed_scale = float(spec.embedding.get("scale", 1.0))
         self.head_name = spec.head["weight"]
         self.embedding = self.head = None
         self.err_flag = None
@@ -144,15 +151,16 @@ class DecoderModel:
         # the residual: float32 [T, H], or [S, T, H] for blocks that keep S streams (each starts as the embedding)
         xs = self.ws.get("residual", (S, T, H), torch.float32)
         self.ws.pending_writeback = None
+        self.ws.pending_entry = None
         self.ws.residual_copy = None
         with phase("embedding"):
             if self.embed_norm is not None:                 # the looked-up rows are normed into the residual
                 raw = self.ws.get("embed_rows", (T, H), torch.float32)
-                K.embedding(batch.tokens, self.embedding, raw, self.err_flag)
+                K.embedding(batch.tokens, self.embedding, raw, self.err_flag, self.embed_scale)
                 self.embed_norm(raw, torch.float32, out=xs[0])
             else:
                 for s in range(S):
-                    K.embedding(batch.tokens, self.embedding, xs[s], self.err_flag)
+                    K.embedding(batch.tokens, self.embedding, xs[s], self.err_flag, self.embed_scale)
         x = xs[0] if S == 1 else xs
         x0 = None
         if self.keep_x0:

@@ -4,3 +4,4 @@ from . import veredra  # noqa: F401
 from . import savenex  # noqa: F401
 from . import nogapel  # noqa: F401
 from . import kikerax  # noqa: F401
+from . import nekorax  # noqa: F401

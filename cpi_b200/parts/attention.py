@@ -41,6 +41,13 @@ lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + c (tensors "lq1", "lk1", "lq2", "lk2"
 rmsnorm(a1 - lambda a2) (1 - c), the norm over the head's values without a weight (`qk_norm_eps`).  A rotation whose
 encoding carries an amplitude multiplies its sines and cosines by it.
 
+Further: `value_rotation` {"theta": base} (the value of position j is turned by j over all its elements, pair m by
+j * base^(-2m / value_dim) in the position part's layout of pairs, and cached so; a head's output at position i is turned
+back by i), `output_gate` "elementwise" (tensor "g" [heads * value_dim, hidden]: the concatenated heads are multiplied by
+sigmoid(g h) element by element; True is the gate per head above), and `sink` {"constant": c} (every head's sink has the
+score c and no tensor: 0 adds one to the softmax denominators).  A mixer without biases, norms, value mixing and
+temperature does its convolution, rotations and cache write in one kernel (`qkv_conv_rotate`) when its sizes allow it.
+
 `attend(...)` below is the choice of the attention kernel for prepared queries and a paged cache; other mixers that
 end in softmax attention over pages (`latent_attention`) call it too.
 """
@@ -48,6 +55,7 @@ from __future__ import annotations
 
 import math
 
+import numpy as np
 import torch
 
 from ..cache.manager import KVRequirement, StateRequirement
@@ -60,6 +68,8 @@ from .linear import MODE_ADD, MODE_STORE, project
 
 # set to False to run every attention through the general kernel (tests compare the two families)
 use_tensor_core_kernels = True
+# set to False to prepare q, k and v with the separate general kernels (tests compare the two)
+use_fused_preparation = True
 
 
 @register_mixer("attention")
@@ -78,7 +88,9 @@ class AttentionMixer(Mixer):
         self.norm_scope = p.get("qk_norm_scope", "head")
         if self.norm_scope not in ("head", "projection"):
             raise ValueError(f"attention: unknown qk_norm_scope '{self.norm_scope}'")
-        self.has_sink = bool(p.get("sink", False))
+        sink = p.get("sink") or False
+        self.has_sink = sink is True
+        self.sink_constant = None if isinstance(sink, bool) else float(sink["constant"])
         rot = p["position"].get("rotary_dims") if p["position"].kind == "rope" else None
         self.rot_dims = self.d if rot is None else int(rot)
         self.taps = None if p.get("conv") is None else int(p["conv"])
@@ -97,14 +109,27 @@ class AttentionMixer(Mixer):
         if self.values_from_keys and self.dv != self.d:
             raise ValueError(f"attention: values that are the keys have the keys' size, not {self.dv} beside {self.d}")
         self.softcap = float(p.get("score_softcap") or 0.0)
-        self.has_gate, self.has_o_bias = bool(p.get("output_gate", False)), bool(p.get("output_bias", False))
+        gate = p.get("output_gate") or False
+        if gate not in (False, True, "elementwise"):
+            raise ValueError(f"attention: unknown output_gate '{gate}'")
+        self.has_gate, self.has_o_bias = bool(gate), bool(p.get("output_bias", False))
+        self.gate_rows = 0 if not gate else self.nh * self.dv if gate == "elementwise" else self.nh
+        self.gate_elementwise = gate == "elementwise"
+        vr = p.get("value_rotation")
+        self.value_theta = None if vr is None else float(vr["theta"])
+        if vr is not None and self.dv % 2:
+            raise ValueError(f"attention: values that turn have an even size, not {self.dv}")
+        if vr is not None and vm is not None:
+            raise ValueError("attention: values that turn are not mixed with another layer's")
         df = p.get("differential")
         self.diff = None if df is None else float(df["lambda_init"])
         self.maps = 1 if self.diff is None else 2
         self.lam = 0.0
-        extended = self.values_from_keys or self.has_gate or self.diff is not None
-        if self.diff is not None and (self.values_from_keys or vm is not None or p.get("sink") or p.get("conv") is not None):
-            raise ValueError("attention: two score maps do not combine with values from keys, value mixing, a sink or a convolution")
+        extended = self.values_from_keys or self.has_gate or self.diff is not None or self.value_theta is not None
+        if self.diff is not None and (self.values_from_keys or vm is not None or sink or p.get("conv") is not None
+                                      or self.gate_elementwise or self.value_theta is not None):
+            raise ValueError("attention: two score maps do not combine with values from keys, value mixing, a sink, a "
+                             "convolution, an elementwise gate or values that turn")
         self.general = (extended or self.bias or self.dv != self.d or self.rot_dims != self.d or self.d % 16 != 0
                         or (bool(p.get("qk_norm", False)) and self.norm_scope == "projection")
                         or self.taps is not None or self.norm_weight_shared or self.value_mix is not None)
@@ -126,6 +151,7 @@ class AttentionMixer(Mixer):
         self.w_qkv = self.w_o = None
         self.rotary = self.score_bias = None
         self.b_qkv = self.w_qnorm = self.w_knorm = self.sink = self.w_conv = self.w_vmix = self.b_o = None
+        self.w_conv_t = self.v_inv_freq = None
         self.keep_first = int(w.get("keep_first") or 0) if self.window_kind == "sliding" else 0
         if self.keep_first < 0:
             raise ValueError(f"attention: keep_first must not be negative, not {self.keep_first}")
@@ -170,7 +196,7 @@ class AttentionMixer(Mixer):
                 if not self.values_from_keys:
                     reqs.append(TensorReq(self.tn["v_bias"], (self.nkv * self.dv,)))
         if self.has_gate:
-            reqs.append(TensorReq(self.tn["g"], (self.nh, self.hidden)))
+            reqs.append(TensorReq(self.tn["g"], (self.gate_rows, self.hidden)))
         if self.has_o_bias:
             reqs.append(TensorReq(self.tn["o_bias"], (self.hidden,)))
         if self.diff is not None:
@@ -237,10 +263,16 @@ class AttentionMixer(Mixer):
         if self.taps is not None:
             names = ["q_conv"] + (["k_conv", "v_conv"] if self.has_kv else [])
             self.w_conv = torch.cat([source.get(self.tn[n], device).to(torch.float32) for n in names], dim=0).contiguous()
+            self.w_conv_t = self.w_conv.t().contiguous()
         if self.value_mix is not None and self.value_mix[0] == "later":
             self.w_vmix = source.get(self.tn["v_mix"], device).to(torch.float32).reshape(1).contiguous()
         if self.has_sink:
             self.sink = source.get(self.tn["sink"], device).to(torch.float32).contiguous()
+        if self.sink_constant is not None:
+            self.sink = torch.full((self.nh,), self.sink_constant, dtype=torch.float32, device=device)
+        if self.value_theta is not None:
+            f = np.float64(self.value_theta) ** (-2.0 * np.arange(self.dv // 2, dtype=np.float64) / self.dv)
+            self.v_inv_freq = torch.from_numpy(f.astype(np.float32)).to(device)
         self.position.prepare(device)
         # what the position part is to this mixer: a rotation of q and k (done with the head norm and the cache
         # write, in one kernel), a bias on the scores (taken by the general attention kernel only), or nothing
@@ -288,11 +320,13 @@ class AttentionMixer(Mixer):
             qkv = self.ws.get("attn_qkv", (T, self.w_qkv.shape[0]), torch.float32)
             with phase("qkv"):
                 project(h, self.w_qkv, qkv)
-            if self.taps is not None:          # the last taps - 1 projected rows of each sequence are its state
-                conv = self.ws.get("attn_qkv_conv", (T, self.w_qkv.shape[0]), torch.float32)
+            qkv_in, gate_in = qkv[:, :self.w_rows()], qkv[:, self.w_rows():]
+            fused = self._fused_preparation(cache)
+            if self.taps is not None and not fused:    # the last taps - 1 projected rows of each sequence are its state
+                conv = self.ws.get("attn_qkv_conv", (T, self.w_rows()), torch.float32)
                 with phase("conv"):
-                    K.causal_conv(qkv, self.w_conv, None, cache.state("conv"), conv, batch, silu=False)
-                qkv = conv
+                    K.causal_conv(qkv_in, self.w_conv, None, cache.state("conv"), conv, batch, silu=False)
+                qkv_in = conv
             v_first, mix_mode = None, 0
             if self.value_mix is not None and cache.owns:
                 v_first = self.ws.get("attn_" + self.value_mix[1], (T, self.nkv * self.dv), torch.float32)
@@ -302,20 +336,28 @@ class AttentionMixer(Mixer):
             if self.maps == 2:
                 q2 = self.ws.get("attn_q2", (T, self.nh * self.d), dt)
                 k2_cache = cache.stream("k2")[0]
+            inv_freq = None if self.rotary is None else self.rotary.inv_freq
+            rot_dims = self.rot_dims if self.rotary is not None else 0
+            interleaved = self.rotary is not None and self.rotary.interleaved
+            amplitude = 1.0 if self.rotary is None else self.rotary.amplitude
             with phase("kv_store"):
-                K.qkv_prepare(qkv, q, k_cache, v_cache, table, page_size, batch.token_seq, batch.token_pos,
-                              batch.seq_slot, n_heads=self.nh, n_kv_heads=self.nkv, head_dim=self.d,
-                              value_dim=self.dv, bias=self.b_qkv, q_norm=self.w_qnorm, k_norm=self.w_knorm,
-                              norm_whole=self.qk_norm and self.norm_scope == "projection",
-                              head_norm=(2 if self.norm_weight_shared else 1) if head_norm else 0,
-                              norm_eps=self.qk_norm_eps,
-                              inv_freq=None if self.rotary is None else self.rotary.inv_freq,
-                              rotary_dims=self.rot_dims if self.rotary is not None else 0,
-                              interleaved=self.rotary is not None and self.rotary.interleaved,
-                              write_kv=self.has_kv and cache.owns, v_first=v_first, v_mix=self.w_vmix,
-                              v_mix_mode=mix_mode, q2_out=q2, k2_cache=k2_cache, values_from_keys=self.values_from_keys,
-                              temperature=self.temperature,
-                              rotary_amplitude=1.0 if self.rotary is None else self.rotary.amplitude)
+                if fused:                       # convolution, rotations and the write into the cache: one kernel
+                    K.qkv_conv_rotate(qkv_in, q, k_cache, v_cache, table, page_size, batch, n_heads=self.nh,
+                                      n_kv_heads=self.nkv, head_dim=self.d, value_dim=self.dv, conv_weight=self.w_conv_t,
+                                      carry=None if self.taps is None else cache.state("conv"), inv_freq=inv_freq,
+                                      rotary_dims=rot_dims, v_inv_freq=self.v_inv_freq, interleaved=interleaved,
+                                      rotary_amplitude=amplitude)
+                else:
+                    K.qkv_prepare(qkv_in, q, k_cache, v_cache, table, page_size, batch.token_seq, batch.token_pos,
+                                  batch.seq_slot, n_heads=self.nh, n_kv_heads=self.nkv, head_dim=self.d,
+                                  value_dim=self.dv, bias=self.b_qkv, q_norm=self.w_qnorm, k_norm=self.w_knorm,
+                                  norm_whole=self.qk_norm and self.norm_scope == "projection",
+                                  head_norm=(2 if self.norm_weight_shared else 1) if head_norm else 0,
+                                  norm_eps=self.qk_norm_eps, inv_freq=inv_freq, rotary_dims=rot_dims,
+                                  interleaved=interleaved, write_kv=self.has_kv and cache.owns, v_first=v_first,
+                                  v_mix=self.w_vmix, v_mix_mode=mix_mode, q2_out=q2, k2_cache=k2_cache,
+                                  values_from_keys=self.values_from_keys, temperature=self.temperature,
+                                  rotary_amplitude=amplitude, v_inv_freq=self.v_inv_freq)
         else:
             qkv = self.ws.get("attn_qkv", (T, self.w_qkv.shape[0]), dt)
             with phase("qkv"):
@@ -335,17 +377,29 @@ class AttentionMixer(Mixer):
             if self.maps == 2:                  # the second map: its own queries and keys, the same values
                 att2 = self.ws.get("attn_out2", (T, self.nh * self.dv), dt)
                 self.attend(q2, att2, k2_cache, v_cache, table, page_size, batch)
-        if att2 is not None or self.has_gate:
+        if self.gate_elementwise or self.v_inv_freq is not None:
+            with phase("head_post"):            # the heads' outputs turned back and gated: one pass
+                gate = gate_in if self.gate_elementwise else None
+                K.head_turn(att, att, batch.token_pos, n_heads=self.nh, value_dim=self.dv, inv_freq=self.v_inv_freq,
+                            interleaved=self.rotary is not None and self.rotary.interleaved, gate=gate)
+        if att2 is not None or (self.has_gate and not self.gate_elementwise):
             with phase("head_post"):            # a1 - lambda a2, its norm, the gate: one pass over the heads' outputs
                 K.head_post(att, att, n_heads=self.nh, value_dim=self.dv, a2=att2, lam=self.lam,
                             norm_eps=self.qk_norm_eps if att2 is not None else None,
                             norm_scale=1.0 if self.diff is None else 1.0 - self.diff,
-                            gate=qkv[:, qkv.shape[1] - self.nh:] if self.has_gate else None)
+                            gate=gate_in if self.has_gate else None)
         with phase("wo"):
             if self.b_o is not None:            # the product adds into rows that hold the bias
                 K.bias_rows(residual, self.b_o, add=add)
                 add = True
             project(att, self.w_o, residual, MODE_ADD if add else MODE_STORE)
+
+    def _fused_preparation(self, cache) -> bool:
+        return (use_fused_preparation and self.has_kv and cache.owns and self.maps == 1 and not self.bias and not self.qk_norm
+                and self.value_mix is None and not self.values_from_keys and self.temperature is None
+                and (self.taps is not None or self.v_inv_freq is not None) and self.w_qkv.shape[0] % 4 == 0
+                and K.qkv_conv_rotate_supported(self.d, self.dv, self.rot_dims if self.rotary is not None else 0,
+                                                self.v_inv_freq is not None, self.taps or 1))
 
     def attend(self, q, att, k_cache, v_cache, table, page_size, batch):
         attend(q, att, k_cache, v_cache, table, page_size, batch, n_heads=self.nh, n_kv_heads=self.nkv, head_dim=self.d,

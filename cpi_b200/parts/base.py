@@ -7,12 +7,15 @@ step's `StepBatch`, and -- for mixers -- the cache and state views the engine ha
 
 Interfaces
 ----------
-Norm          requirements(); load(src, dev); __call__(x, out_dtype, rows=None) -> tensor
+Norm          requirements(); load(src, dev); __call__(x, out_dtype, rows=None) -> tensor;
+              enter(y, x, following, h_out)             # x += norm(y); h_out = following(x)
 Position      (no weights) prepare(dev); encoding() -> RotaryEncoding | ScoreBias | None, consumed by its mixer
 Mixer         requirements(); load(src, dev); kv_requirement(); state_requirements();
               forward(h, residual, batch, cache)        # residual += mixer(h)
-FeedForward   requirements(); load(src, dev); forward(h, residual, batch)   # residual += ffn(h)
-Block         run(layer, residual, batch, cache)        # the arrangement of the above
+FeedForward   requirements(); load(src, dev); forward(h, residual, batch)   # residual += ffn(h);
+              a routed one may also have expert_sum(h, batch) -> ExpertSum | None: its output, not yet added up
+Block         run(layer, residual, batch, cache)        # the arrangement of the above; a block that norms the sublayers'
+              outputs as well as their inputs declares two more norms (LayerSpec.mixer_post_norm, feed_forward_post_norm)
 Junction      requirements(); load(src, dev); run(x, x0, batch)   # between two layers: rewrites the residual x in
               place; x0 is the embedding output (kept by the model when a junction sets `needs_embedding_output`)
 
@@ -55,6 +58,36 @@ class Part:
 class Norm(Part):
     def __call__(self, x, out_dtype, rows=None, out=None):
         raise NotImplementedError
+
+    def enter(self, y, x, following=None, h_out=None):
+        """x += norm(y) for a sublayer's output y (float32 rows or an ExpertSum), then h_out = following(x) if given."""
+        raise NotImplementedError(f"{type(self).__name__} does not norm a sublayer's output")
+
+
+@dataclass(frozen=True)
+class ExpertSum:
+    """The output of routed experts before it is added up: per token the sum, in the order of its choices, of the chosen
+    experts' output rows y[row_of_slot] (already weighted), or of weight * h for a chosen expert number >= n_real (an
+    expert whose output is its input).  Lives in workspace buffers until the same part runs again."""
+    y: torch.Tensor                # float32 [rows, width]
+    row_of_slot: torch.Tensor      # int32 [T, k]
+    expert: torch.Tensor           # int32 [T, k]
+    weight: torch.Tensor           # float32 [T, k]
+    h: torch.Tensor                # [T, width], the experts' input
+    n_real: int
+
+    def lists(self):
+        return self.y, self.row_of_slot, self.expert, self.weight, self.h, self.n_real
+
+    def add_to(self, x, add=True):
+        """x (+)= the sums."""
+        from ..csrc import lib as K
+        K.norm_step(x, experts=self.lists(), add=add)
+
+    def rows(self, ws):
+        out = ws.get("expert_sum", (self.h.shape[0], self.y.shape[-1]), torch.float32)
+        self.add_to(out, add=False)
+        return out
 
 
 @dataclass(frozen=True)

@@ -21,6 +21,11 @@ adds it into the float32 residual and writes the next sublayer's input; the copy
 next layer's input when that layer is of this kind too.  A mixer that is a weighted sum of branches hands its branches
 over (`branch_outputs`), so that the sum, the norm and the addition are one pass.
 
+"sandwich_norm": x += norm1b(mixer(norm1(x))); x += norm2b(ffn(norm2(x))): a norm before and one after every sublayer
+(the layer's mixer_norm / feed_forward_norm and mixer_post_norm / feed_forward_post_norm, of any kinds).  The entry of a
+sublayer's output into the residual and the norm before the next sublayer are one kernel when both norms act element by
+element; the entry of a layer's last sublayer is left to the next layer's first kernel (`Workspace.pending_entry`).
+
 "scaled_pre_norm": x += m * mixer(norm1(x)); x += m * ffn(norm2(x)) with one constant m (`residual_scale`).  It is the
 arrangement above with a single stream and constant coefficients (read 1, mix 1, write m), so the scaled addition of a
 sublayer's output rides on the kernel that forms the next sublayer's normed input.
@@ -130,6 +135,8 @@ class HyperConnectionsBlock(Block):
         T, H = x.shape[1], x.shape[2]
         ws = layer.mixer_norm.ws
         before, ws.pending_writeback = ws.pending_writeback, None
+        if ws.pending_entry is not None:
+            ws.settle()
         if before is not None and before[0].data_ptr() != x.data_ptr():
             ws.pending_writeback = before          # another residual's: not ours to fuse
             ws.settle()
@@ -229,3 +236,46 @@ class PostNormBlock(Block):
         y = ws.get("post_norm_y", (T, H), torch.float32)
         HyperConnectionsBlock._run_part(layer.feed_forward, h, y, batch)
         self._enter(ws, [y], [1.0], layer.feed_forward_norm, x, batch.dtype)
+
+
+@register_block("sandwich_norm")
+class SandwichNormBlock(Block):
+    """No params and no tensors of its own."""
+    graph_safe = True
+
+    def __init__(self, spec, prefix="", **_):
+        super().__init__(spec, prefix)
+
+    def run(self, layer, residual, batch, cache):
+        # (the products of these chains stay on the single-CTA kernel, as the post_norm block's do and for its reason)
+        with single_cta_products():
+            self._run(layer, residual, batch, cache)
+
+    def _run(self, layer, x, batch, cache):
+        ws = layer.mixer_norm.ws
+        if x.dim() != 2:
+            raise ValueError("sandwich_norm: the block keeps one residual stream")
+        T, H = x.shape
+        before, ws.pending_entry = ws.pending_entry, None
+        if before is not None and before[0].data_ptr() != x.data_ptr():
+            ws.pending_entry, before = before, None
+        ws.settle()
+        h = ws.get("norm_mixer", (T, H), batch.dtype)
+        with phase("rmsnorm"):
+            if before is None:
+                layer.mixer_norm(x, batch.dtype, out=h)
+            else:
+                before[2].enter(before[1], x, layer.mixer_norm, h)
+        y = ws.get("sandwich_y", (T, H), torch.float32)
+        HyperConnectionsBlock._run_part(layer.mixer, h, y, batch, cache)
+        if layer.feed_forward is None:
+            ws.pending_entry = (x, y, layer.mixer_post_norm)
+            return
+        h2 = ws.get("norm_ffn", (T, H), batch.dtype)
+        with phase("rmsnorm"):
+            layer.mixer_post_norm.enter(y, x, layer.feed_forward_norm, h2)
+        out = getattr(layer.feed_forward, "expert_sum", lambda *a: None)(h2, batch)
+        if out is None:
+            out = ws.get("sandwich_y", (T, H), torch.float32)
+            HyperConnectionsBlock._run_part(layer.feed_forward, h2, out, batch)
+        ws.pending_entry = (x, out, layer.feed_forward_post_norm)

@@ -17,10 +17,14 @@ moe_swiglu    params: hidden_size, num_experts, top_k, expert_size, shared_size 
               made on s + choice bias (`router_rule` {"choice_bias": a tensor name [E] or None, "groups": n, "keep": m,
               "scale": c}; only experts of the m best of n equal groups of neighbours can be chosen, a group's score
               being the sum of its two largest choice scores), and the chosen experts' outputs are weighted by their s
-              divided by the chosen s' sum, times c), router_bias (a tensor name [E] added to the logits,
+              divided by the chosen s' sum, times c | "scored": the same with the choices in `router_rule`: "score"
+              ("sigmoid", or "softmax" over all of a token's logits), "group_score" ("top2_sum" or "max"), "normalise" (the
+              division by the chosen scores' sum)), router_bias (a tensor name [E] added to the logits,
               or None), expert_layout ("stacked", below, or "per_expert": `expert_names` {"gate", "up", "down"} with
               "{e}" for the expert's number, each [out, in]), router_name, shared (None or the params of a
-              dense_swiglu part that runs for every token beside the routed experts, instead of shared_size)
+              dense_swiglu part that runs for every token beside the routed experts, instead of shared_size),
+              activation ("silu", "gelu_tanh" or "swish_clamped" with `limit`, as above), identity_experts (n: the router
+              knows n more experts, after the others, whose output is the input h itself; they have no tensors)
               tensors: feed_forward.router.weight [E, H], feed_forward.experts.gate_up_proj [E, H, 2I],
               feed_forward.experts.down_proj [E, I, H], feed_forward.shared_expert.{gate,up,down}_proj.weight
 
@@ -39,7 +43,7 @@ import torch
 from ..csrc import lib as K
 from ..phases import active as phases_active, phase
 from ..weights.store import TensorReq
-from .base import FeedForward, register_feed_forward
+from .base import ExpertSum, FeedForward, register_feed_forward
 from .linear import (MODE_ADD, MODE_CLAMPED_GLU, MODE_GEGLU, MODE_STORE, MODE_STORE_GELU, MODE_STORE_RELU2, MODE_SWIGLU,
                      project)
 
@@ -154,26 +158,41 @@ class MoESwiGLU(FeedForward):
         self.hidden, self.n_experts, self.top_k = int(p["hidden_size"]), int(p["num_experts"]), int(p["top_k"])
         self.inter, self.shared_inter = int(p["expert_size"]), int(p.get("shared_size", 0))
         self.gate_mode = p.get("router_gate", "sigmoid_input")
-        if self.gate_mode not in ("sigmoid_input", "sigmoid_output", "none", "softmax_chosen", "sigmoid_normed"):
+        if self.gate_mode not in ("sigmoid_input", "sigmoid_output", "none", "softmax_chosen", "sigmoid_normed", "scored"):
             raise ValueError(f"moe_swiglu: unknown router_gate '{self.gate_mode}'")
+        self.activation, self.limit = p.get("activation", "silu"), float(p.get("limit") or 0.0)
+        if self.activation not in K.GATE_ACTS:
+            raise ValueError(f"moe_swiglu: unknown activation '{self.activation}'; known: {sorted(K.GATE_ACTS)}")
+        if self.activation == "swish_clamped" and not self.limit > 0:
+            raise ValueError("moe_swiglu: the clamped activation needs a positive limit")
+        self.n_identity = int(p.get("identity_experts") or 0)
+        self.n_routed = self.n_experts + self.n_identity           # what the router chooses from
+        if self.n_identity < 0 or (self.n_identity and self.gate_mode in ("sigmoid_input", "none")):
+            raise ValueError("moe_swiglu: identity experts go with a gate on the experts' outputs")
         rule = dict(p.get("router_rule") or {})
         self.rule = None
         self.n_choice_bias = None
-        if self.gate_mode == "sigmoid_normed":
+        if self.gate_mode in ("sigmoid_normed", "scored"):
             groups, keep = int(rule.get("groups", 1)), int(rule.get("keep", 1))
-            if not (1 <= keep <= groups <= 64) or int(p["num_experts"]) % groups:
-                raise ValueError(f"moe_swiglu: {p['num_experts']} experts in {groups} groups of which {keep} are kept")
-            if int(p["top_k"]) > keep * (int(p["num_experts"]) // groups):
+            if not (1 <= keep <= groups <= 64) or self.n_routed % groups:
+                raise ValueError(f"moe_swiglu: {self.n_routed} experts in {groups} groups of which {keep} are kept")
+            if int(p["top_k"]) > keep * (self.n_routed // groups):
                 raise ValueError(f"moe_swiglu: top_k {p['top_k']} exceeds the experts of the {keep} kept groups")
             self.rule = {"choice_bias": None, "groups": groups, "keep": keep, "scale": float(rule.get("scale", 1.0))}
+            if self.gate_mode == "scored":
+                self.rule.update(score=rule.get("score", "sigmoid"), group_score=rule.get("group_score", "top2_sum"),
+                                 normalise=bool(rule.get("normalise", True)))
+                if self.rule["score"] not in ("sigmoid", "softmax") or self.rule["group_score"] not in ("top2_sum", "max"):
+                    raise ValueError(f"moe_swiglu: unknown score '{self.rule['score']}' or group_score "
+                                     f"'{self.rule['group_score']}'")
             if rule.get("choice_bias") is not None:
                 self.n_choice_bias = prefix + rule["choice_bias"]
         elif rule:
-            raise ValueError("moe_swiglu: router_rule belongs to the gate 'sigmoid_normed'")
-        if not 1 <= self.top_k <= self.n_experts:
-            raise ValueError(f"moe_swiglu: top_k {self.top_k} of {self.n_experts} experts")
-        if self.n_experts > 256:
-            raise ValueError(f"moe_swiglu: {self.n_experts} experts (supported: up to 256)")
+            raise ValueError("moe_swiglu: router_rule belongs to the gates 'sigmoid_normed' and 'scored'")
+        if not 1 <= self.top_k <= self.n_routed:
+            raise ValueError(f"moe_swiglu: top_k {self.top_k} of {self.n_routed} experts")
+        if self.n_routed > 256:
+            raise ValueError(f"moe_swiglu: {self.n_routed} experts (supported: up to 256)")
         self.ws = workspace
         f = prefix + "feed_forward."
         self.n_router, self.n_gate_up, self.n_down = f + "router.weight", f + "experts.gate_up_proj", f + "experts.down_proj"
@@ -211,11 +230,11 @@ class MoESwiGLU(FeedForward):
         self.capture = None        # a list: every forward appends a copy of its expert choices [T, k]
 
     def requirements(self):
-        reqs = [TensorReq(self.n_router, (self.n_experts, self.hidden))]
+        reqs = [TensorReq(self.n_router, (self.n_routed, self.hidden))]
         if self.n_router_bias is not None:
-            reqs.append(TensorReq(self.n_router_bias, (self.n_experts,)))
+            reqs.append(TensorReq(self.n_router_bias, (self.n_routed,)))
         if self.n_choice_bias is not None:
-            reqs.append(TensorReq(self.n_choice_bias, (self.n_experts,)))
+            reqs.append(TensorReq(self.n_choice_bias, (self.n_routed,)))
         if self.layout == "per_expert":
             for e in range(self.n_experts):
                 reqs += [TensorReq(self.expert_names["gate"].format(e=e), (self.inter, self.hidden)),
@@ -246,8 +265,16 @@ class MoESwiGLU(FeedForward):
         if self.shared is not None:
             self.shared.load(source, device)
 
+    def expert_sum(self, h, batch):
+        """The routed experts' outputs before they are added up (see ExpertSum), for a block that does more with the sum
+        than add it to the residual; None when a shared expert adds to it as well."""
+        return None if self.shared is not None else self._run(h, None, batch, defer=True)
+
     def forward(self, h, residual, batch):
-        T, E, Kk = h.shape[0], self.n_experts, self.top_k
+        self._run(h, residual, batch)
+
+    def _run(self, h, residual, batch, defer=False):
+        T, E, R, Kk = h.shape[0], self.n_experts, self.n_routed, self.top_k
         ws, i32, f32 = self.ws, torch.int32, torch.float32
         forked = None
         if self.shared is not None and self.overlap_shared and h.is_cuda and phases_active() is None:
@@ -262,8 +289,8 @@ class MoESwiGLU(FeedForward):
                 forked.record(self._side_stream)
         idx = ws.get("moe_topk_idx", (T, Kk), i32)
         gate = ws.get("moe_topk_gate", (T, Kk), f32)
-        logits = ws.get("moe_router_logits", (T, E), f32)
-        offsets = ws.get("moe_offsets", (E + 1,), i32)
+        logits = ws.get("moe_router_logits", (T, R), f32)
+        offsets = ws.get("moe_offsets", (R + 1,), i32)
         row_token = ws.get("moe_row_token", (T * Kk,), i32)
         row_scale = ws.get("moe_row_scale", (T * Kk,), f32)
         row_of_slot = ws.get("moe_row_of_slot", (T * Kk,), i32)
@@ -274,33 +301,36 @@ class MoESwiGLU(FeedForward):
         with phase("moe_router"):
             gathered = K.moe_route(h, self.w_router, idx, gate, logits, offsets, row_token, row_scale, row_of_slot,
                                    top_k=Kk, sorted_h=sorted_h, bias=self.b_router,
-                                   sigmoid_gate=self.gate_mode if self.gate_mode in ("softmax_chosen", "sigmoid_normed")
+                                   sigmoid_gate=self.gate_mode if self.gate_mode in ("softmax_chosen", "sigmoid_normed", "scored")
                                    else self.gate_mode != "none", rule=self.rule)
         if self.capture is not None:
             self.capture.append(idx.clone())
-        hint = max(1, -(-M // E))
+        # identity experts come after the others, so their rows are the last ones and lie outside the products' E groups
+        hint = max(1, -(-M // R))
+        offsets = offsets[:E + 1]
+        act_mode = {"silu": MODE_SWIGLU, "gelu_tanh": MODE_GEGLU, "swish_clamped": MODE_CLAMPED_GLU}[self.activation]
         act = ws.get("moe_act", (M, self.inter), h.dtype)
         in_scale = row_scale if self.gate_mode == "sigmoid_input" else None
         with phase("moe_expert"):
             if sortable:
                 if not gathered:
                     K.gather_rows(h, row_token, sorted_h)
-                project(sorted_h, self.w_gate_up, act, MODE_SWIGLU, m_rows=M, row_scale=in_scale,
+                project(sorted_h, self.w_gate_up, act, act_mode, m_rows=M, row_scale=in_scale, gate_limit=self.limit,
                         group_offsets=offsets, n_groups=E, rows_per_group_hint=hint)
             else:
-                project(h, self.w_gate_up, act, MODE_SWIGLU, m_rows=M, a_rows=row_token, row_scale=in_scale,
-                        group_offsets=offsets, n_groups=E, rows_per_group_hint=hint)
-            out_scale = row_scale if self.gate_mode in ("sigmoid_output", "softmax_chosen", "sigmoid_normed") else None
+                project(h, self.w_gate_up, act, act_mode, m_rows=M, a_rows=row_token, row_scale=in_scale,
+                        gate_limit=self.limit, group_offsets=offsets, n_groups=E, rows_per_group_hint=hint)
+            out_scale = row_scale if self.gate_mode in ("sigmoid_output", "softmax_chosen", "sigmoid_normed", "scored") else None
             # One expert per token: the down projection can add straight into the residual rows.  Beside a shared
             # expert on the second stream that needs an order (two kernels adding into the same rows at once would
             # sum in whatever order they meet): in a step with many tokens the join comes before the down
             # projection (each product fills the GPU by itself, so nothing is lost by the wait, and the stored
             # outputs and the combine kernel go); in a step with few tokens the two chains run side by side to the
             # end and the combine adds the routed outputs after the join.
-            join_early = forked is not None and Kk == 1 and T >= self.join_early_tokens
+            join_early = forked is not None and Kk == 1 and T >= self.join_early_tokens and not self.n_identity
             if join_early:
                 torch.cuda.current_stream().wait_event(forked)
-            direct = Kk == 1 and (forked is None or join_early)
+            direct = Kk == 1 and (forked is None or join_early) and not defer and not self.n_identity
             if direct:
                 project(act, self.w_down, residual, MODE_ADD, m_rows=M, out_rows=row_token, row_scale=out_scale,
                         group_offsets=offsets, n_groups=E, rows_per_group_hint=hint)
@@ -308,11 +338,16 @@ class MoESwiGLU(FeedForward):
                 y = ws.get("moe_y", (M, self.hidden), f32)
                 project(act, self.w_down, y, MODE_STORE, m_rows=M, row_scale=out_scale,
                         group_offsets=offsets, n_groups=E, rows_per_group_hint=hint)
+        if defer:
+            return ExpertSum(y, row_of_slot, idx, gate, h, E)
         if not direct:
             if forked is not None:
                 torch.cuda.current_stream().wait_event(forked)
             with phase("moe_merge"):
-                K.moe_combine(residual, y, row_of_slot, top_k=Kk)
+                if self.n_identity:
+                    ExpertSum(y, row_of_slot, idx, gate, h, E).add_to(residual)
+                else:
+                    K.moe_combine(residual, y, row_of_slot, top_k=Kk)
         if forked is not None:
             return
         if self.shared is not None:

@@ -2,7 +2,10 @@
 
 "concat_linear"  x <- W [x ; x0]: the residual and the embedding output side by side (x first) through one matrix
                  W [width, 2 width].  params: hidden_size, weight (tensor name).  The operand row is formed in the
-                 activation dtype; the product accumulates in float32 and writes the float32 residual.
+                 activation dtype; the product accumulates in float32 and writes the float32 residual.  With `step`
+                 (tensor name, [times, width]) and `pass_index` t: x <- W [x ; x0] + step[t], for a range of layers that
+                 runs several times and marks its passes; junctions that name the same matrix share one copy of it.
+                 `products` "single_cta": the product stays on the single-CTA kernel (see `single_cta_products`).
 
 "token_gated_input"  x <- x + rmsnorm(P (gelu_tanh(G x) * e)) * w: every token brings a small vector e of its own, the
                  columns [offset, offset + dim) of its row in a table indexed by token id (one table may serve many
@@ -15,13 +18,30 @@
 """
 from __future__ import annotations
 
+import contextlib
+
 import torch
 
 from ..csrc import lib as K
 from ..phases import phase
 from ..weights.store import TensorReq
 from .base import Junction, register_junction
-from .linear import project
+from .linear import MODE_ADD, project, single_cta_products
+
+
+def shared_tensor(source, name, device):
+    """The named tensor on the device, one copy for all the parts that are loaded from the same source."""
+    shared = getattr(source, "_shared_tables", None)
+    if shared is None:
+        shared = {}
+        try:
+            source._shared_tables = shared
+        except AttributeError:
+            pass
+    key = (name, str(device))
+    if key not in shared:
+        shared[key] = source.get(name, device).contiguous()
+    return shared[key]
 
 
 @register_junction("concat_linear")
@@ -33,19 +53,33 @@ class ConcatLinear(Junction):
         super().__init__(spec, prefix)
         self.hidden = int(spec["hidden_size"])
         self.weight_name = prefix + spec["weight"]
-        self.ws, self.weight = workspace, None
+        self.step_name = None if spec.get("step") is None else prefix + spec["step"]
+        self.pass_index, self.passes = int(spec.get("pass_index", 0)), int(spec.get("passes", 1))
+        if not 0 <= self.pass_index < self.passes:
+            raise ValueError(f"concat_linear: pass {self.pass_index} of {self.passes}")
+        self.single_cta = spec.get("products") == "single_cta"
+        self.ws, self.weight, self.step = workspace, None, None
 
     def requirements(self):
-        return [TensorReq(self.weight_name, (self.hidden, 2 * self.hidden))]
+        reqs = [TensorReq(self.weight_name, (self.hidden, 2 * self.hidden))]
+        if self.step_name is not None:
+            reqs.append(TensorReq(self.step_name, (self.passes, self.hidden)))
+        return reqs
 
     def load(self, source, device):
-        self.weight = source.get(self.weight_name, device).contiguous()
+        self.weight = shared_tensor(source, self.weight_name, device)
+        if self.step_name is not None:
+            self.step = source.get(self.step_name, device)[self.pass_index].to(torch.float32).contiguous()
 
     def run(self, x, x0, batch) -> None:
         cat = self.ws.get("junction_cat", (x.shape[0], 2 * self.hidden), batch.dtype)
-        with phase("junction"):
+        with phase("junction"), (single_cta_products() if self.single_cta else contextlib.nullcontext()):
             K.concat_rows(x, x0, cat)
-            project(cat, self.weight, x)
+            if self.step is None:
+                project(cat, self.weight, x)
+            else:                                  # the product adds into rows that hold the pass's vector
+                K.bias_rows(x, self.step)
+                project(cat, self.weight, x, MODE_ADD)
 
 
 @register_junction("token_gated_input")
@@ -72,17 +106,7 @@ class TokenGatedInput(Junction):
 
     def load(self, source, device):
         n = self.names
-        shared = getattr(source, "_shared_tables", None)      # one copy on the device for the layers of one source
-        if shared is None:
-            shared = {}
-            try:
-                source._shared_tables = shared
-            except AttributeError:
-                pass
-        key = (n["table"], str(device))
-        if key not in shared:
-            shared[key] = source.get(n["table"], device).contiguous()
-        self.table = shared[key]
+        self.table = shared_tensor(source, n["table"], device)
         gate, proj = source.get(n["gate"], device), source.get(n["proj"], device)
         dt = torch.float32 if torch.float32 in (gate.dtype, proj.dtype) else torch.bfloat16
         self.w_gate, self.w_proj = gate.to(dt).contiguous(), proj.to(dt).contiguous()

@@ -7,7 +7,9 @@
                      learned sink per head (its exponential joins the denominator, without a key or a value);
                      out = W_o concat_heads(sum_j p_j value_j).
                      params: hidden_size, heads, head_dim (plain), rot_dim, value_dim, q_rank, kv_rank, softmax_scale,
-                     norm_eps, position (PartSpec; a rotation of rot_dim elements, or "none"), sink (bool),
+                     norm_eps, position (PartSpec; a rotation of rot_dim elements, or "none"; its amplitude multiplies the
+                     sines and cosines of both rotated parts), sink (bool), window (None, {"kind": "full"} or {"kind":
+                     "sliding", "size": n}: a position sees itself and the n - 1 before it),
                      tensor_names {"dq", "dq_norm", "uq", "dkv", "dkv_norm", "uk", "uv", "o", "sink"}.
                      cache: one stream "latent" of one head of kv_rank + rot_dim elements per position.
 
@@ -52,6 +54,13 @@ class LatentAttentionMixer(Mixer):
         self.q_rank, self.kv_rank = int(p["q_rank"]), int(p["kv_rank"])
         self.scale, self.eps = float(p["softmax_scale"]), float(p["norm_eps"])
         self.has_sink = bool(p.get("sink", False))
+        w = p.get("window") or {"kind": "full"}
+        if w["kind"] not in ("full", "sliding"):
+            raise ValueError(f"latent_attention: a window of kind '{w['kind']}' (full or sliding)")
+        self.window_kind = w["kind"]
+        self.window = int(w["size"]) if w["kind"] == "sliding" else 0
+        if w["kind"] == "sliding" and self.window < 1:
+            raise ValueError(f"latent_attention: a window of {self.window} positions")
         self.row = self.kv_rank + self.r              # what a position keeps, and the size of a query head
         if self.r % 2 or self.r < 0:
             raise ValueError(f"latent_attention: a rotated part of {self.r} elements (an even number)")
@@ -104,7 +113,7 @@ class LatentAttentionMixer(Mixer):
                              f"part has {self.r}")
 
     def kv_requirement(self):
-        return KVRequirement(1, self.row, "full", 0, streams=(("latent", 1, self.row),))
+        return KVRequirement(1, self.row, self.window_kind, self.window, streams=(("latent", 1, self.row),))
 
     def forward(self, h, residual, batch, cache, add=True):
         T, f32, dt = h.shape[0], torch.float32, h.dtype
@@ -112,12 +121,13 @@ class LatentAttentionMixer(Mixer):
         pages, table, page_size = cache.stream("latent")
         inv_freq = None if self.rotary is None else self.rotary.inv_freq
         inter = self.rotary is not None and self.rotary.interleaved
+        amp = 1.0 if self.rotary is None else self.rotary.amplitude
         down = self.ws.get("latent_down", (T, self.q_rank + row), f32)
         with phase("qkv"):
             project(h, self.w_down, down)
         with phase("kv_store"):          # the normed latent and the rotated key part of every token go into its page
             K.latent_kv_write(down[:, self.q_rank:], self.w_cnorm, self.eps, inv_freq, inter, pages, table, page_size,
-                              batch.token_seq, batch.token_pos, batch.seq_slot, rank=rank, rot=R)
+                              batch.token_seq, batch.token_pos, batch.seq_slot, rank=rank, rot=R, amplitude=amp)
         cq = self.ws.get("latent_cq", (T, self.q_rank), dt)
         with phase("rmsnorm"):
             K.rmsnorm(down[:, :self.q_rank], self.w_qnorm, self.eps, cq)
@@ -130,7 +140,7 @@ class LatentAttentionMixer(Mixer):
         rows = self.ws.get("latent_rows", (H * T,), torch.int32)
         with phase("kv_store"):
             K.latent_q_split(q, inv_freq, inter, plain, full, offsets, rows, batch.token_pos, n_heads=H, dim=D, rot=R,
-                             rank=rank)
+                             rank=rank, amplitude=amp)
         with phase("qkv"):               # the plain part of every query through its head's W_uk^T, into full[t, head, :rank]
             project(plain, self.w_ukT, full.view(T * H, row)[:, :rank], MODE_STORE, out_rows=rows, group_offsets=offsets,
                     n_groups=H, rows_per_group_hint=T)
@@ -141,21 +151,22 @@ class LatentAttentionMixer(Mixer):
                 if batch.is_decode:
                     # key splits from a bucketed bound of the context, so that a captured graph keeps its shape
                     groups = -(-H // 64)
-                    tiles = -(-batch.ctx_bucket // K.LATENT_KEY_TILE)
+                    keys = batch.ctx_bucket if not self.window else min(batch.ctx_bucket, self.window + K.LATENT_KEY_TILE)
+                    tiles = -(-keys // K.LATENT_KEY_TILE)
                     n_splits = max(1, min(K.sm_count() // max(1, T * groups), tiles // 2,
                                           K.latent_attention_max_splits()))
                     K.latent_attention(full, lat, pages, table, page_size, batch.token_seq, batch.token_pos,
                                        batch.seq_slot, n_heads=H, rank=rank, scale=self.scale, sink=self.sink,
-                                       n_splits=n_splits)
+                                       n_splits=n_splits, window=self.window)
                 else:
                     K.latent_attention(full, lat, pages, table, page_size, batch.token_seq, batch.token_pos,
                                        batch.seq_slot, n_heads=H, rank=rank, scale=self.scale, sink=self.sink,
-                                       tile_tok0=batch.tile_tok0, tile_rows=batch.tile_rows)
+                                       tile_tok0=batch.tile_tok0, tile_rows=batch.tile_rows, window=self.window)
         else:
             att = self.ws.get("latent_att", (T, H * row), dt)
             with phase("latent_attention"):
                 attend(full, att, pages, pages, table, page_size, batch, n_heads=H, n_kv_heads=1, head_dim=row,
-                       value_dim=row, window_kind="full", window_size=0, scale=self.scale, sink=self.sink)
+                       value_dim=row, window_kind=self.window_kind, window_size=self.window, scale=self.scale, sink=self.sink)
             with phase("wo"):
                 K.head_major_rows(att, lat, n_heads=H, n=rank)
         with phase("wo"):
