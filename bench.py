@@ -48,6 +48,10 @@ same way.
 soft-capped attention over its own keys and a gated linear recurrent unit; norms on the sublayers' outputs; gelu
 feed-forwards and experts chosen from the best groups) at two layer sizes beside Savenex's layers (attention beside a
 gated delta rule, dense and routed feed-forwards) at the same sizes, measured the same way.
+`--workload nekorax`: the Nekorax design (attention with short convolutions, values that turn with their positions and an
+elementwise gate alternating with windowed attention over a cached latent; tanh norms before and after every sublayer;
+clamped and identity experts chosen from the best groups; a pass entered through a matrix) at two layer sizes beside
+Nogapel's layers (mixers) and Kikerax's (experts, norms on the outputs) at the same sizes, measured the same way.
 """
 from __future__ import annotations
 
@@ -1124,6 +1128,137 @@ def run_kikerax(args) -> dict:
     return out
 
 
+NEKORAX_SIZES = {
+    # width, attention (heads, kv heads, head size = value size, taps), latent (heads, plain, rotated, value, query rank,
+    # latent rank, window), experts (count, identity ones besides, top, ff each, groups, kept): two points with the layer
+    # shapes of 1-3 B and 7-8 B parameter models
+    "w2048": dict(width=2048, attn=(16, 4, 128, 4), latent=(16, 128, 64, 128, 768, 512, 1024), moe=(16, 4, 4, 1024, 4, 3)),
+    "w4096": dict(width=4096, attn=(32, 8, 128, 4), latent=(32, 128, 64, 128, 1536, 512, 1024), moe=(16, 4, 4, 2048, 4, 3)),
+}
+
+
+def nekorax_config(sz: dict, vocab: int, pairs: int) -> dict:
+    """(attention, latent attention) x pairs, every layer with routed experts; the first pair is entered as a pass."""
+    H, G, D, taps = sz["attn"]
+    lh, ld, lr, lv, qr, kr, win = sz["latent"]
+    E, ident, top, eff, groups, keep = sz["moe"]
+    mlp = {"kind": "moe", "expert": {"ff": eff, "limit": 7.0},
+           "router": {"experts": E, "identity": ident, "top": top, "groups": {"count": groups, "keep": keep}}}
+    pair = [{"type": "attention", "mlp": mlp,
+             "mixer": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "conv": taps, "rot": {"base": 1e6, "dims": D // 2}}},
+            {"type": "latent_attention", "mlp": mlp,
+             "mixer": {"heads": lh, "dim": ld, "rot_dim": lr, "vdim": lv, "q_rank": qr, "kv_rank": kr, "scale": (ld + lr) ** -0.5,
+                       "mask": {"size": win}, "rot": {"base": 1e4, "dims": lr, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0,
+                                                                                           "slow": 1.0}}}}]
+    return {"architecture": "Nekorax", "layers": pair * pairs, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "vocab": vocab,
+            "width": sz["width"], "logit_softcap": 30.0, "loop": {"start": 0, "stop": 2, "times": 1}}
+
+
+def nogapel_like_nekorax_config(sz: dict, vocab: int, pairs: int) -> dict:
+    """The closest model the library had for the mixers: Nogapel layers (attention with the same convolution, latent
+    attention) at the same head counts, sizes and ranks; both see everything; a small dense feed-forward."""
+    H, G, D, taps = sz["attn"]
+    lh, ld, lr, lv, qr, kr, _ = sz["latent"]
+    mlp = {"kind": "dense", "ff": sz["width"]}
+    pair = [{"type": "attention", "mlp": mlp,
+             "mixer": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "conv": taps, "v_mix": True,
+                       "rot": {"base": 1e6, "dims": D // 2}}},
+            {"type": "latent_attention", "mlp": mlp,
+             "mixer": {"heads": lh, "dim": ld, "rot_dim": lr, "vdim": lv, "q_rank": qr, "kv_rank": kr, "scale": (ld + lr) ** -0.5,
+                       "rot": {"base": 1e4, "dims": lr}}}]
+    return {"architecture": "Nogapel", "layers": pair * pairs, "norm": {"eps": 1e-6}, "vocab": vocab, "width": sz["width"]}
+
+
+def kikerax_like_nekorax_config(sz: dict, vocab: int, layers: int) -> dict:
+    """The closest model the library had for the experts and for norms on the sublayers' outputs: Kikerax layers with as
+    many experts of the same size per token, chosen from the best groups, without a shared expert."""
+    H, G, D, _ = sz["attn"]
+    E, _, top, eff, groups, _ = sz["moe"]
+    one = {"type": "attention",
+           "mlp": {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": E, "top": top, "groups": {"count": groups, "keep": 2}}},
+           "mixer": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "diff": 0.5, "rot": {"base": 1e6, "dims": D // 2}}}
+    return {"architecture": "Kikerax", "layers": [one] * layers, "norm": {"eps": 1e-6}, "vocab": vocab, "width": sz["width"],
+            "logit_softcap": 30.0}
+
+
+def run_nekorax(args) -> dict:
+    """Prefill and decode of Nekorax at two layer sizes, with the time of every phase per layer that has it and each
+    phase's share of its roofline, beside the like phases of Nogapel layers (mixers) and Kikerax layers (experts, norms on
+    the outputs) at equal sizes: products by flops over the measured bf16 rate in prefill and by weight bytes over the
+    measured copy rate in decode; attention by flops / cache bytes; row kernels by bytes."""
+    import torch
+
+    pk = peaks()
+    vocab, T, B, pairs = 32000, 2048, 8, 2
+    n_layers = 2 * pairs
+    g = torch.Generator().manual_seed(7)
+    toks = lambda n: torch.randint(0, vocab, (n,), generator=g).tolist()
+    out = {"metric": "tokens/s, Nekorax beside Nogapel and Kikerax layers at equal layer sizes (bf16, random weights)",
+           "unit": "tokens/s", "dtype": "bf16", "data": "synthetic", "peaks": pk, "points": {}}
+    tf, bw = pk["bf16_tflops"] * 1e12, pk["hbm_gbs"] * 1e9
+    sizes = {k: v for k, v in NEKORAX_SIZES.items() if not args.sizes or k in args.sizes.split(",")}
+    for name, sz in sizes.items():
+        W = sz["width"]
+        H, G, D, taps = sz["attn"]
+        lh, ld, lr, lv, qr, kr, win = sz["latent"]
+        E, ident, top, eff, _, _ = sz["moe"]
+        runs = {"nekorax": measure_config(nekorax_config(sz, vocab, pairs), vocab, T, B, toks),
+                "nogapel": measure_config(nogapel_like_nekorax_config(sz, vocab, pairs), vocab, T, B, toks),
+                "kikerax": measure_config(kikerax_like_nekorax_config(sz, vocab, n_layers), vocab, T, B, toks)}
+
+        def frac(model, phases, per, prefill, decode):
+            """`prefill`, `decode`: (flops, bytes) of the phases in one layer; `per`: layers that have them."""
+            res = {}
+            for step, (flops, nbytes), key in (("prefill", prefill, "prefill"), ("decode", decode, "decode_per_step")):
+                ms = sum(runs[model]["phases_ms"][key].get(n, 0) for n in phases) / per
+                res[step] = None if not ms else round(max(flops / tf, nbytes / bw) / (ms / 1e3), 4)
+            return res
+
+        ctx = T - 64
+        keys_all, keys_win = T * (T + 1) // 2, sum(min(t + 1, win) for t in range(T))
+        row = kr + lr
+        a_in = (H + 2 * G) * D
+        a_proj, g_proj = (a_in + H * D) * W, H * D * W                            # q, k, v, o; the gate's rows
+        l_proj = (qr + row) * W + qr * lh * (ld + lr) + lh * ld * kr + lh * kr * lv + lh * lv * W
+        att = ((4.0 * D * H * keys_all, 0.0), (0.0, B * ctx * G * 2 * D * 2.0))
+        lat = lambda keys, seen: ((2.0 * lh * keys * (row + kr), 0.0), (2.0 * B * lh * seen * (row + kr), B * seen * row * 2.0))
+        proj = lambda n: ((2.0 * T * n, 0.0), (0.0, 2.0 * n))
+        rows = lambda nbytes: ((0.0, T * nbytes), (0.0, B * nbytes))
+        chosen = top * E / (E + ident)                                            # chosen experts with matrices, per token
+        touched = lambda k: E * (1.0 - (1.0 - k / E) ** B)
+        moe = lambda k: ((2.0 * T * 3.0 * W * k * eff, 0.0), (0.0, 2.0 * touched(k) * 3.0 * W * eff))
+        latent_rows = (qr + row) * 4.0 + lh * (ld + lr) * (4.0 + 2.0) + row * 2.0
+        roof = {
+            "attention (a constant sink; tensor-core kernels both)": {
+                "nekorax": frac("nekorax", ["attention"], pairs, *att), "nogapel": frac("nogapel", ["attention"], pairs, *att)},
+            "attention over the cached latent (windowed / over everything)": {
+                "nekorax": frac("nekorax", ["latent_attention"], pairs, *lat(keys_win, win)),
+                "nogapel": frac("nogapel", ["latent_attention"], pairs, *lat(keys_all, ctx))},
+            "mixer projections in and out": {
+                "nekorax": frac("nekorax", ["qkv", "wo"], pairs, *proj(a_proj + g_proj + l_proj)),
+                "nogapel": frac("nogapel", ["qkv", "wo"], pairs, *proj(a_proj + l_proj))},
+            "row kernels of the mixers (convolution, rotations, cache write, outputs turned back and gated / convolution, head norm, rotation, value mixing, cache write)": {
+                "nekorax": frac("nekorax", ["kv_store", "conv", "head_post"], pairs, *rows(a_in * (4 + 2.0) + H * D * (2 + 2 + 4.0) + latent_rows)),
+                "nogapel": frac("nogapel", ["kv_store", "conv"], pairs, *rows(a_in * (4 + 4 + 4 + 2.0) + latent_rows))},
+            "routed experts (router, lists, products; kikerax: with the combination)": {
+                "nekorax": frac("nekorax", ["moe_router", "moe_expert"], n_layers, *moe(chosen)),
+                "kikerax": frac("kikerax", ["moe_router", "moe_expert", "moe_merge"], n_layers, *moe(top))},
+            "norms and the residual (nekorax: the combination of the experts' outputs, four norms and two sums in two kernels, and the latent's query norm; kikerax: one kernel per sublayer)": {
+                "nekorax": frac("nekorax", ["rmsnorm"], n_layers,
+                                *rows(W * ((4 + 4 + 4 + 2.0) + (chosen * 4 + 2 + 4 + 4 + 2.0)) + qr * (4 + 2.0) / 2)),
+                "kikerax": frac("kikerax", ["rmsnorm"], n_layers, *rows(2 * W * (4 + 4 + 4 + 2.0)))},
+            "entry of a pass (concatenation, product, vector; no like kernel)": {
+                "nekorax": frac("nekorax", ["junction"], 1, *((2.0 * T * 2 * W * W, T * W * (8 + 4 + 4 + 8.0)), (0.0, 4.0 * W * W)))},
+        }
+        out["points"][name] = {"sizes": sz, "layers": n_layers, "prefill_tokens": T, "decode_batch": B, "decode_context": ctx,
+                               **runs, "fraction_of_roofline": roof}
+    big = out["points"][sorted(out["points"])[-1]]
+    out["value"] = big["nekorax"]["decode_tok_s"]
+    out["config"] = {"model": "Nekorax, (attention, windowed latent attention) x 2, routed and identity experts in every layer",
+                     "global_batch": B, "seq_len": T, "parallelism": "single GPU", "l2": "weights of a step exceed the L2"}
+    return out
+
+
 def reference_arm_reason() -> str:
     """Why `--impl reference` has nothing to run, as found on this image (one line)."""
     return ("kurulav1/cpi is a CMake C++/CUDA project (no setup.py or pyproject.toml, so pip has nothing to install); "
@@ -1143,8 +1278,9 @@ def main() -> int:
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--context", type=int, default=4096)
     ap.add_argument("--skip-points", action="store_true")
-    ap.add_argument("--sizes", default="", help="--workload nogapel | kikerax: a comma-separated subset of its size points")
-    ap.add_argument("--workload", choices=["scout24", "maverick4", "long131k", "contexts", "cpu_baseline", "veredra", "savenex", "nogapel", "kikerax"],
+    ap.add_argument("--sizes", default="", help="--workload nogapel | kikerax | nekorax: a comma-separated subset of its size points")
+    ap.add_argument("--workload", choices=["scout24", "maverick4", "long131k", "contexts", "cpu_baseline", "veredra", "savenex", "nogapel", "kikerax",
+                                               "nekorax"],
                     default="scout24")
     ap.add_argument("--reference-root", default=os.environ.get("CPI_REFERENCE_ROOT"),
                     help="a checkout of kurulav1/cpi (for --workload cpu_baseline)")
@@ -1167,6 +1303,9 @@ def main() -> int:
         return 0
     if args.workload == "kikerax":
         print(json.dumps(run_kikerax(args)))
+        return 0
+    if args.workload == "nekorax":
+        print(json.dumps(run_nekorax(args)))
         return 0
     if args.workload == "nogapel":
         print(json.dumps(run_nogapel(args)))
