@@ -152,109 +152,125 @@ struct SelectRule {
 
 // One warp per token; lane l holds experts l, l + 32, ...  Every comparison takes the lower index at a tie and never a
 // NaN, and every sum has one order, so a token's choice depends on its logits alone.
-__device__ __forceinline__ void warp_best(float& v, int& i) {      // the largest v, ties to the lowest i; i < 0: nothing
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    const float ov = __shfl_xor_sync(0xffffffffu, v, o);
-    const int oi = __shfl_xor_sync(0xffffffffu, i, o);
-    if (oi >= 0 && (i < 0 || ov > v || (ov == v && oi < i))) { v = ov; i = oi; }
-  }
+//
+// A choice score as an unsigned number of the same order (0: nothing); -0 counts as 0.
+__device__ __forceinline__ unsigned order_key(float v) {
+  const int b = __float_as_int(v + 0.0f);
+  return (unsigned)b ^ ((unsigned)(b >> 31) | 0x80000000u);
+}
+__device__ __forceinline__ float key_value(unsigned k) {
+  return __uint_as_float(k & 0x80000000u ? k ^ 0x80000000u : ~k);
+}
+// the index of the warp's largest key, the lowest at a tie; -1 when no lane has one
+__device__ __forceinline__ int warp_best(unsigned& key, int i) {
+  const unsigned best = __reduce_max_sync(0xffffffffu, key);
+  const unsigned at = __reduce_min_sync(0xffffffffu, key == best ? (unsigned)i : 0xffffffffu);
+  key = best;
+  return best == 0u ? -1 : (int)at;
 }
 
 __device__ __forceinline__ void select_scored_warp(const float* lg, int* idx, float* gate, int n_experts, int top_k,
                                                    const SelectRule& r) {
   constexpr int PER = kMaxExperts / 32;
-  const int lane = threadIdx.x & 31;
-  float s[PER], c[PER];
+  const int lane = threadIdx.x & 31, nj = (n_experts + 31) >> 5;      // registers in use (the same for the whole warp)
+  float s[PER];
+  unsigned key[PER];                     // of the choice score; 0: cannot be chosen (any more)
   if (r.flavour & kScoreSoftmax) {
     float mx = -INFINITY, sum = 0.f;
 #pragma unroll
-    for (int j = 0; j < PER; ++j) {
-      const int e = lane + 32 * j;
-      s[j] = e < n_experts ? lg[e] : -INFINITY;
-      mx = fmaxf(mx, s[j]);
-    }
+    for (int j = 0; j < PER; ++j)
+      if (j < nj) {
+        const int e = lane + 32 * j;
+        s[j] = e < n_experts ? lg[e] : -INFINITY;
+        mx = fmaxf(mx, s[j]);
+      }
     mx = warp_max(mx);
 #pragma unroll
-    for (int j = 0; j < PER; ++j) { s[j] = lane + 32 * j < n_experts ? expf(s[j] - mx) : 0.f; sum += s[j]; }
+    for (int j = 0; j < PER; ++j)
+      if (j < nj) { s[j] = lane + 32 * j < n_experts ? expf(s[j] - mx) : 0.f; sum += s[j]; }
     sum = warp_sum(sum);
 #pragma unroll
-    for (int j = 0; j < PER; ++j) s[j] /= sum;
+    for (int j = 0; j < PER; ++j)
+      if (j < nj) s[j] /= sum;
   } else {
 #pragma unroll
-    for (int j = 0; j < PER; ++j) { const int e = lane + 32 * j; s[j] = e < n_experts ? 1.0f / (1.0f + expf(-lg[e])) : 0.f; }
+    for (int j = 0; j < PER; ++j)
+      if (j < nj) { const int e = lane + 32 * j; s[j] = e < n_experts ? 1.0f / (1.0f + expf(-lg[e])) : 0.f; }
   }
 #pragma unroll
   for (int j = 0; j < PER; ++j) {
+    key[j] = 0u;
     const int e = lane + 32 * j;
-    c[j] = e < n_experts && r.choice_bias ? s[j] + r.choice_bias[e] : s[j];
+    if (j < nj && e < n_experts) {
+      const float c = r.choice_bias ? s[j] + r.choice_bias[e] : s[j];
+      if (c == c) key[j] = order_key(c);
+    }
   }
-  unsigned open = 0;                     // bit j: expert lane + 32 j can (still) be chosen
-  const int per = n_experts / r.n_groups;
-#pragma unroll
-  for (int j = 0; j < PER; ++j) open |= (lane + 32 * j < n_experts && c[j] == c[j]) ? 1u << j : 0u;
   if (r.n_groups > 1 && r.keep_groups < r.n_groups) {
-    // lane g and lane g + 32 hold the scores of groups g and g + 32 (up to 64)
-    float gs[2] = {-INFINITY, -INFINITY};
+    const int per = n_experts / r.n_groups;
+    int grp[PER];
+#pragma unroll
+    for (int j = 0; j < PER; ++j)
+      if (j < nj) grp[j] = (lane + 32 * j) / per;
+    // lane g holds the scores of groups g and g + 32 (up to 64)
+    unsigned gk[2] = {0u, 0u};
+    const int passes = (r.flavour & kGroupLargest) || per < 2 ? 1 : 2;
     for (int g = 0; g < r.n_groups; ++g) {
       float total = 0.f;
       int first = -1;
-      for (int pass = 0; pass < ((r.flavour & kGroupLargest) || per < 2 ? 1 : 2); ++pass) {
-        float v = -INFINITY;
-        int i = -1;
+      for (int pass = 0; pass < passes; ++pass) {
+        unsigned k = 0u;
+        int i = 0;
 #pragma unroll
-        for (int j = 0; j < PER; ++j) {
-          const int e = lane + 32 * j;
-          if (((open >> j) & 1u) && e / per == g && e != first && (i < 0 || c[j] > v)) { v = c[j]; i = e; }
-        }
-        warp_best(v, i);
+        for (int j = 0; j < PER; ++j)
+          if (j < nj && grp[j] == g && lane + 32 * j != first && key[j] > k) { k = key[j]; i = lane + 32 * j; }
+        first = warp_best(k, i);
+        const float v = first < 0 ? -INFINITY : key_value(k);
         total = pass == 0 ? v : total + v;
-        first = i;
       }
-      if ((g & 31) == lane) gs[g >> 5] = total;
+      if (g == lane) gk[0] = order_key(total);
+      if (g == lane + 32) gk[1] = order_key(total);
     }
     unsigned long long kept = 0ull;
-    for (int k = 0; k < r.keep_groups; ++k) {
-      float v = 0.f;
-      int i = -1;
-#pragma unroll
-      for (int u = 0; u < 2; ++u) {
-        const int g = lane + 32 * u;
-        if (g < r.n_groups && !((kept >> g) & 1ull) && (i < 0 || gs[u] > v)) { v = gs[u]; i = g; }
-      }
-      warp_best(v, i);
-      kept |= 1ull << i;
+    for (int n = 0; n < r.keep_groups; ++n) {
+      const bool low = gk[0] >= gk[1];
+      unsigned k = low ? gk[0] : gk[1];
+      const int g = warp_best(k, low ? lane : lane + 32);
+      kept |= 1ull << g;
+      if (g == lane) gk[0] = 0u;
+      if (g == lane + 32) gk[1] = 0u;
     }
 #pragma unroll
     for (int j = 0; j < PER; ++j)
-      if (lane + 32 * j < n_experts && !((kept >> ((lane + 32 * j) / per)) & 1ull)) open &= ~(1u << j);
+      if (j < nj && key[j] && !((kept >> grp[j]) & 1ull)) key[j] = 0u;
   }
   float sum = 0.f;
   unsigned taken = 0;
-  for (int k = 0; k < top_k; ++k) {
-    float v = 0.f, sc = 0.f;
-    int i = -1;
+  for (int n = 0; n < top_k; ++n) {
+    unsigned k = 0u;
+    int i = 0;
 #pragma unroll
     for (int j = 0; j < PER; ++j)
-      if (((open >> j) & 1u) && (i < 0 || c[j] > v)) { v = c[j]; i = lane + 32 * j; }
-    warp_best(v, i);
+      if (j < nj && key[j] > k) { k = key[j]; i = lane + 32 * j; }
+    i = warp_best(k, i);
     if (i < 0) {                         // nothing left to choose from: the lowest free index
-      int f = n_experts;
+      unsigned f = 0xffffffffu;
 #pragma unroll
       for (int j = PER - 1; j >= 0; --j)
         if (lane + 32 * j < n_experts && !((taken >> j) & 1u)) f = lane + 32 * j;
-      i = -__reduce_max_sync(0xffffffffu, -f);
+      i = (int)__reduce_min_sync(0xffffffffu, f);
     }
+    float sc = 0.f;
 #pragma unroll
     for (int j = 0; j < PER; ++j)
-      if (lane + 32 * j == i) { open &= ~(1u << j); taken |= 1u << j; sc = s[j]; }
+      if (j < nj && lane + 32 * j == i) { key[j] = 0u; taken |= 1u << j; sc = s[j]; }
     sc = __shfl_sync(0xffffffffu, sc, i & 31);
-    if (lane == 0) { idx[k] = i; gate[k] = sc; }
+    if (lane == 0) { idx[n] = i; gate[n] = sc; }
     sum += sc;
   }
   const float f = r.flavour & kWeightsAsScored ? r.gate_scale : r.gate_scale / (sum + 1e-20f);
   if (lane == 0)
-    for (int k = 0; k < top_k; ++k) gate[k] *= f;
+    for (int n = 0; n < top_k; ++n) gate[n] *= f;
 }
 
 // The k best logits of one token, ties to the lowest index; gate = 1 (mode 0), the sigmoid of the chosen logit
@@ -383,58 +399,73 @@ moe_route_small_kernel(const float* __restrict__ logits, int n_tokens, int n_exp
 //   row_token[m]              token whose activation feeds logical row m
 //   row_scale[m]              gate of that (token, k)
 //   row_of_slot[t*K + k]      logical row that holds (t, k)'s expert output
-// A warp owns experts warp, warp + 32, ...; it scans the slots 32 at a time and places the matching
-// ones with a ballot, which keeps them in slot order.
-constexpr int kListSlotsInSmem = 8192;
+// A warp owns a run of consecutive slots and looks at them 32 at a time: lanes with the same expert find each other
+// (match), so a slot's place is its expert's rows before this warp's run, plus those earlier in the run, plus the lanes
+// below it.  Two passes: the first counts per warp and expert, the second places; both keep the slots' order.
 __global__ void __launch_bounds__(1024)
 moe_lists_kernel(const int* __restrict__ topk_idx, const float* __restrict__ topk_gate,
                  int* __restrict__ group_offsets, int* __restrict__ row_token,
                  float* __restrict__ row_scale, int* __restrict__ row_of_slot,
                  int n_slots, int top_k, int n_experts) {
   pdl_launch_dependents();
-  pdl_wait();
-  __shared__ int counts[kMaxExperts];
+  __shared__ int rows_s[32 * kMaxExperts];            // [warp][expert]: counts, then the next row
   __shared__ int offsets[kMaxExperts + 1];
-  __shared__ int idx_s[kListSlotsInSmem];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  // the choices are scanned twice by every warp: keep them in shared memory when they fit
-  const bool staged = n_slots <= kListSlotsInSmem;
-  if (staged) {
-    for (int s = threadIdx.x; s < n_slots; s += blockDim.x) idx_s[s] = topk_idx[s];
-    __syncthreads();
+  for (int i = threadIdx.x; i < 32 * n_experts; i += 1024) rows_s[i] = 0;
+  const int run = ((n_slots + 1023) / 1024) * 32;     // slots of a warp, a multiple of 32
+  const int begin = warp * run, end = min(n_slots, begin + run);
+  int* mine = rows_s + warp * n_experts;
+  __syncthreads();
+  pdl_wait();
+  for (int s0 = begin; s0 < end; s0 += 32) {
+    const int s = s0 + lane;
+    const int e = s < end ? topk_idx[s] : -1;
+    const unsigned peers = __match_any_sync(0xffffffffu, e);
+    if (e >= 0 && lane == __ffs(peers) - 1) mine[e] += __popc(peers);
+    __syncwarp();
   }
-  const int* idx = staged ? idx_s : topk_idx;
-  for (int e = warp; e < n_experts; e += 32) {
-    int c = 0;
-    for (int s0 = 0; s0 < n_slots; s0 += 32) {
-      const int s = s0 + lane;
-      const bool hit = s < n_slots && idx[s] == e;
-      c += __popc(__ballot_sync(0xffffffffu, hit));
+  __syncthreads();
+  for (int e = threadIdx.x; e < n_experts; e += 1024) {      // counts -> rows of the expert before each warp's run
+    int before = 0;
+    for (int w = 0; w < 32; ++w) {
+      const int c = rows_s[w * n_experts + e];
+      rows_s[w * n_experts + e] = before;
+      before += c;
     }
-    if (lane == 0) counts[e] = c;
+    offsets[e + 1] = before;
   }
   __syncthreads();
-  if (threadIdx.x == 0) {
-    int run = 0;
-    for (int i = 0; i < n_experts; ++i) { offsets[i] = run; run += counts[i]; }
-    offsets[n_experts] = run;
-  }
-  __syncthreads();
-  for (int e = threadIdx.x; e <= n_experts; e += blockDim.x) group_offsets[e] = offsets[e];
-  for (int e = warp; e < n_experts; e += 32) {
-    int m = offsets[e];
-    for (int s0 = 0; s0 < n_slots; s0 += 32) {
-      const int s = s0 + lane;
-      const bool hit = s < n_slots && idx[s] == e;
-      const unsigned mask = __ballot_sync(0xffffffffu, hit);
-      if (hit) {
-        const int r = m + __popc(mask & ((1u << lane) - 1u));
-        row_token[r] = s / top_k;
-        row_scale[r] = topk_gate[s];
-        row_of_slot[s] = r;
+  if (warp == 0) {                                           // running sum over the experts, 32 at a time
+    int carry = 0;
+    for (int e0 = 0; e0 < n_experts; e0 += 32) {
+      int v = e0 + lane < n_experts ? offsets[e0 + lane + 1] : 0;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int u = __shfl_up_sync(0xffffffffu, v, o);
+        if (lane >= o) v += u;
       }
-      m += __popc(mask);
+      v += carry;
+      if (e0 + lane < n_experts) offsets[e0 + lane + 1] = v;
+      carry = __shfl_sync(0xffffffffu, v, 31);
     }
+    if (lane == 0) offsets[0] = 0;
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e <= n_experts; e += 1024) group_offsets[e] = offsets[e];
+  for (int s0 = begin; s0 < end; s0 += 32) {
+    const int s = s0 + lane;
+    const int e = s < end ? topk_idx[s] : -1;
+    const unsigned peers = __match_any_sync(0xffffffffu, e);
+    int r = 0;
+    if (e >= 0) {
+      r = offsets[e] + mine[e] + __popc(peers & ((1u << lane) - 1u));
+      row_token[r] = s / top_k;
+      row_scale[r] = topk_gate[s];
+      row_of_slot[s] = r;
+    }
+    __syncwarp();
+    if (e >= 0 && lane == __ffs(peers) - 1) mine[e] += __popc(peers);
+    __syncwarp();
   }
 }
 
