@@ -7,7 +7,7 @@
 //   qkv_conv_rotate   per token, from float32 projection rows [q | k | v]: a causal convolution over time of every
 //                     channel (optional; inputs before the step's first token come from the sequence's carried inputs),
 //                     the rotation of q and k, the rotation of v (optional), q to its buffer, k and v into the cache
-//                     pages.  A thread owns eight columns (four pairs) and walks over up to 16 consecutive tokens of one
+//                     pages.  A thread owns eight columns (four pairs) and walks over a few consecutive tokens of one
 //                     sequence with the convolution's last inputs in registers, so every input is read once; the block's
 //                     sines and cosines are computed once per (token, pair) for all its heads.  In a step of single
 //                     tokens the same launch also updates the carried inputs (nobody else reads or writes those columns).
@@ -20,7 +20,7 @@
 
 namespace cpi {
 
-constexpr int QR_THREADS = 128, QR_TB = 16, QR_MAX_PAIRS = 128;
+constexpr int QR_THREADS = 128, QR_MAX_TB = 32, QR_MAX_PAIRS = 128, QR_BLOCKS_PER_SM = 4;
 
 struct ConvRotParams {
   const float* qkv; long stride;                   // [T, >= C], C = NH D + NKV D + NKV DV
@@ -33,6 +33,7 @@ struct ConvRotParams {
   const int* page_table; int max_blocks; int page_size;
   const int* token_seq; const int* token_pos; const int* seq_slot; const int* seq_start;
   const int* tile_tok0; const int* tile_rows; int subs;      // null: a tile is one token
+  int tb;                                          // tokens of a block
   int n_heads, n_kv_heads, head_dim, v_dim;
 };
 
@@ -79,17 +80,17 @@ __device__ __forceinline__ void group_columns(int g, int rot, int interleaved, i
 }
 
 template <typename TO, int TAPS>
-__global__ void __launch_bounds__(QR_THREADS) qkv_conv_rotate_kernel(ConvRotParams p) {
+__global__ void __launch_bounds__(QR_THREADS, TAPS > 4 ? 2 : QR_BLOCKS_PER_SM) qkv_conv_rotate_kernel(ConvRotParams p) {
   pdl_launch_dependents();
-  extern __shared__ float table_s[];               // [QR_TB][pairs] cosines then sines: of q and k, then of v
-  __shared__ size_t kv_row_s[QR_TB];
-  const int tid = threadIdx.x;
+  extern __shared__ float table_s[];               // [tb][pairs] cosines then sines: of q and k, then of v
+  __shared__ size_t kv_row_s[QR_MAX_TB];
+  const int tid = threadIdx.x, TB = p.tb;
   int tok0, ntok;
   if (p.tile_tok0) {
-    const int tile = blockIdx.x / p.subs, off = (blockIdx.x % p.subs) * QR_TB, rows = p.tile_rows[tile];
+    const int tile = blockIdx.x / p.subs, off = (blockIdx.x % p.subs) * TB, rows = p.tile_rows[tile];
     if (off >= rows) return;
     tok0 = p.tile_tok0[tile] + off;
-    ntok = min(QR_TB, rows - off);
+    ntok = min(TB, rows - off);
   } else {
     tok0 = blockIdx.x;
     ntok = 1;
@@ -99,7 +100,7 @@ __global__ void __launch_bounds__(QR_THREADS) qkv_conv_rotate_kernel(ConvRotPara
   const int rp = p.inv_freq ? p.rot_dims >> 1 : 0, vp = p.v_inv_freq ? DV >> 1 : 0;
   const int c0 = blockIdx.y * QR_THREADS * 8, c1 = min(C, c0 + QR_THREADS * 8);      // the block's columns, as groups of 8
   float* qk_t = table_s;
-  float* v_t = table_s + 2 * QR_TB * rp;
+  float* v_t = table_s + 2 * TB * rp;
   const int seq = p.token_seq[tok0], slot = p.seq_slot[seq];
   // positions and tables are on the device before the step's first kernel: nothing here waits for the projection
   if (c0 < nq + nk)
@@ -108,7 +109,7 @@ __global__ void __launch_bounds__(QR_THREADS) qkv_conv_rotate_kernel(ConvRotPara
       float s, c;
       sincosf((float)p.token_pos[tok0 + t] * p.inv_freq[m], &s, &c);
       qk_t[t * rp + m] = c * p.amplitude;
-      qk_t[(QR_TB + t) * rp + m] = s * p.amplitude;
+      qk_t[(TB + t) * rp + m] = s * p.amplitude;
     }
   if (c1 > nq + nk)
     for (int i = tid; i < ntok * vp; i += QR_THREADS) {
@@ -116,7 +117,7 @@ __global__ void __launch_bounds__(QR_THREADS) qkv_conv_rotate_kernel(ConvRotPara
       float s, c;
       sincosf((float)p.token_pos[tok0 + t] * p.v_inv_freq[m], &s, &c);
       v_t[t * vp + m] = c;
-      v_t[(QR_TB + t) * vp + m] = s;
+      v_t[(TB + t) * vp + m] = s;
     }
   if (tid < ntok) {
     const int pos = p.token_pos[tok0 + tid];
@@ -169,15 +170,23 @@ __global__ void __launch_bounds__(QR_THREADS) qkv_conv_rotate_kernel(ConvRotPara
       hist[j][4] = b.x; hist[j][5] = b.y; hist[j][6] = b.z; hist[j][7] = b.w;
     }
   }
+  // the columns of the next two tokens are asked for before a token's work
   const float* src = p.qkv + (size_t)tok0 * p.stride;
-  float4 na = *reinterpret_cast<const float4*>(src + colA), nb = *reinterpret_cast<const float4*>(src + colB);
+  float4 na[2], nb[2];
+#pragma unroll
+  for (int u = 0; u < 2; ++u) {
+    const float* at = src + (size_t)min(u, ntok - 1) * p.stride;
+    na[u] = *reinterpret_cast<const float4*>(at + colA);
+    nb[u] = *reinterpret_cast<const float4*>(at + colB);
+  }
 #pragma unroll 1
   for (int t = 0; t < ntok; ++t) {
-    const float in[8] = {na.x, na.y, na.z, na.w, nb.x, nb.y, nb.z, nb.w};
-    if (t + 1 < ntok) {                            // the next token's columns are asked for before this one's work
-      src += p.stride;
-      na = *reinterpret_cast<const float4*>(src + colA);
-      nb = *reinterpret_cast<const float4*>(src + colB);
+    const float in[8] = {na[0].x, na[0].y, na[0].z, na[0].w, nb[0].x, nb[0].y, nb[0].z, nb[0].w};
+    na[0] = na[1]; nb[0] = nb[1];
+    if (t + 2 < ntok) {
+      const float* at = src + (size_t)(t + 2) * p.stride;
+      na[1] = *reinterpret_cast<const float4*>(at + colA);
+      nb[1] = *reinterpret_cast<const float4*>(at + colB);
     }
     float v[8];
 #pragma unroll
@@ -199,7 +208,7 @@ __global__ void __launch_bounds__(QR_THREADS) qkv_conv_rotate_kernel(ConvRotPara
 #pragma unroll
       for (int i = 0; i < 8; ++i) hist[TAPS > 1 ? TAPS - 2 : 0][i] = in[i];
     }
-    if (pair >= 0) turn4(v, tab + t * np + pair, tab + (QR_TB + t) * np + pair, p.interleaved, 1.0f);
+    if (pair >= 0) turn4(v, tab + t * np + pair, tab + (TB + t) * np + pair, p.interleaved, 1.0f);
     TO* dst;
     if (is_q) dst = reinterpret_cast<TO*>(p.q_out) + ((size_t)(tok0 + t) * p.n_heads + head) * D;
     else dst = reinterpret_cast<TO*>(is_v ? p.v_cache : p.k_cache) + (kv_row_s[t] + (size_t)head * p.page_size) * dim;
@@ -357,10 +366,22 @@ extern "C" int cpi_qkv_conv_rotate(const float* qkv, long stride, const float* c
   const long C = (long)n_heads * head_dim + (long)n_kv_heads * (head_dim + v_dim);
   ConvRotParams p{qkv, stride, conv_wt, taps, carry, tile_tok0 == nullptr, inv_freq, inv_freq ? rot_dims : 0, v_inv_freq,
                   interleaved, amplitude, q_out, k_cache, v_cache, page_table, max_blocks, page_size, token_seq, token_pos,
-                  seq_slot, seq_start, tile_tok0, tile_rows, (max_tile_rows + QR_TB - 1) / QR_TB, n_heads, n_kv_heads,
-                  head_dim, v_dim};
-  const dim3 grid(tile_tok0 ? n_tiles * p.subs : n_tokens, (unsigned)((C / 8 + QR_THREADS - 1) / QR_THREADS));
-  const size_t smem = 2 * QR_TB * ((inv_freq ? rot_dims / 2 : 0) + (v_inv_freq ? v_dim / 2 : 0)) * sizeof(float);
+                  seq_slot, seq_start, tile_tok0, tile_rows, 1, 1, n_heads, n_kv_heads, head_dim, v_dim};
+  const int by = (int)((C / 8 + QR_THREADS - 1) / QR_THREADS);
+  if (tile_tok0) {
+    // tokens of a block: what makes the fewest (waves of blocks) x (tokens, and the inputs before the first one)
+    const long slots = (long)sm_count() * QR_BLOCKS_PER_SM;
+    long best = -1;
+    const long pairs = (inv_freq ? rot_dims / 2 : 0) + (v_inv_freq ? v_dim / 2 : 0);
+    for (int tb = 4; tb <= QR_MAX_TB && 2 * tb * pairs * (long)sizeof(float) <= 48 * 1024; ++tb) {      // (four always fit)
+      const long blocks = (long)n_tiles * ((max_tile_rows + tb - 1) / tb) * by;
+      const long cost = ((blocks + slots - 1) / slots) * (tb + taps + 1);
+      if (best < 0 || cost < best) { best = cost; p.tb = tb; }
+    }
+    p.subs = (max_tile_rows + p.tb - 1) / p.tb;
+  }
+  const dim3 grid(tile_tok0 ? n_tiles * p.subs : n_tokens, by);
+  const size_t smem = 2 * p.tb * ((inv_freq ? rot_dims / 2 : 0) + (v_inv_freq ? v_dim / 2 : 0)) * sizeof(float);
 #define CPI_QR(TO, TAPS) cpi::launch_pdl(qkv_conv_rotate_kernel<TO, TAPS>, grid, dim3(QR_THREADS), smem, stream, p)
   // one tap is a product with one weight: it runs as a convolution of four taps with three zeros
   CPI_DISPATCH_DTYPE(out_dtype, TO, {

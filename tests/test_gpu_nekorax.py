@@ -261,7 +261,7 @@ def _pages(T, page, n_pages, seed):
 
 @pytest.mark.parametrize("H,G,D,Dv,dims,taps,inter", [(4, 2, 64, 64, 32, 4, False), (6, 2, 16, 8, 8, 3, False), (2, 1, 24, 40, 16, 8, True),
                                                       (1, 1, 8, 8, 8, 1, False), (2, 2, 128, 128, 64, 2, True), (3, 1, 10, 14, 6, 3, False),
-                                                      (2, 1, 32, 64, 0, 5, False), (5, 1, 16, 16, 8, None, True)])
+                                                      (2, 1, 32, 64, 0, 5, False), (5, 1, 16, 16, 8, None, True), (1, 1, 256, 256, 256, 2, False)])
 def test_preparation_with_convolution_and_values_that_turn(H, G, D, Dv, dims, taps, inter):
     """Rows [q | k | v | rest]: convolution, rotation of q and k, rotation of the values by their positions, into pages --
     the fused kernel where its sizes allow it, and the separate ones always: a sequence of 80 tokens whole, in portions
