@@ -24,7 +24,7 @@ MAX_DECODE_SPLITS = 256          # key splits that the combine kernel of decode 
 GENERAL_ATTENTION_MAX_DIM = 640  # largest key or value row of the general attention kernel
 PREFILL_TILE_ROWS = 256          # most query rows of one sequence that a block of the prefill attention kernel takes
 
-ABI_VERSION = 6                  # what cpi_abi_version() of a matching library answers
+ABI_VERSION = 7                  # what cpi_abi_version() of a matching library answers
 
 _lib = None
 scratch_generation = 0    # grows whenever a scratch buffer of this module is (re)allocated
@@ -501,6 +501,34 @@ def norm_step(x, *, y=None, experts=None, post=None, pre=None, h_out=None, rows=
           c_int(n), c_int(W), _stream())
 
 
+def rms_step(x, *, y=None, experts=None, post, pre=None, h_out=None, add=True):
+    """One boundary between sublayers with RMS norms on both sides: x (float32 [T, W], in place) (+)= post(v), v being the
+    row y[t] (float32) or the sum over a token's chosen experts (`experts`: as in `norm_step`); then, with `pre`, h_out =
+    pre(x).  A norm is (weight [W], offset, eps): v / sqrt(mean(v^2) + eps) * (offset + weight)."""
+    _need_cuda(x, y, h_out, post[0])
+    T, W = x.shape
+    assert x.dtype == torch.float32 and x.stride(1) == 1 and (y is None) != (experts is None) and (pre is None) == (h_out is None)
+    assert y is None or (y.dtype == torch.float32 and y.shape == (T, W) and y.stride(1) == 1)
+    ye = ros = idx = wt = h = None
+    top_k = n_real = 0
+    if experts is not None:
+        ye, ros, idx, wt, h, n_real = experts
+        _need_cuda(ye, ros, idx, wt, h)
+        top_k = idx.shape[-1]
+        assert ye.dtype == torch.float32 and ye.is_contiguous() and ye.shape[-1] == W and h.shape == (T, W) and h.stride(1) == 1
+        assert ros.dtype == idx.dtype == torch.int32 and wt.dtype == torch.float32
+        assert ros.numel() == idx.numel() == wt.numel() == T * top_k and ros.is_contiguous() and idx.is_contiguous()
+    assert h_out is None or (h_out.shape == (T, W) and h_out.stride(1) == 1)
+    for norm in (post, pre):
+        assert norm is None or (norm[0].is_cuda and norm[0].is_contiguous() and norm[0].numel() == W)
+    b = pre or (None, 0.0, 0.0)
+    code = lambda t: c_int(F32 if t is None else dtype_code(t.dtype))
+    _call("cpi_rms_step", _p(y), c_long(0 if y is None else y.stride(0)), _p(ye), _p(ros), _p(idx), _p(wt), _p(h), code(h),
+          c_long(0 if h is None else h.stride(0)), c_int(top_k), c_int(n_real), _p(x), c_long(x.stride(0)), c_int(int(add)),
+          _p(post[0]), code(post[0]), c_float(post[1]), c_float(post[2]), _p(b[0]), code(b[0]), c_float(b[1]), c_float(b[2]),
+          _p(h_out), code(h_out), c_long(0 if h_out is None else h_out.stride(0)), c_int(T), c_int(W), _stream())
+
+
 def sum_norm_add(branches, scales, weight, out, *, eps=0.0, add=True, h_out=None, normalise=True):
     """out (+)= rmsnorm(sum_b scales[b] * branches[b]) * weight over rows: up to four float32 [T, W] branches with a
     constant each, one norm over their sum (`normalise` False: the scaled sum as it is); `h_out` (any dtype, [T, W])
@@ -699,14 +727,25 @@ def causal_conv(x, weight, bias, carry, out, batch, *, silu=True, in_bias=None):
 
 def linear_scan(k, q, v, state, out, batch, *, n_heads, heads_per_group, n_rows, n_cols, z=None, z_bias=None,
                 tau=1.0, dt=None, dt_bias=None, a_log=None, skip=None, q_scale=1.0, decay_ready=False,
-                decay_kind=0, beta=None):
+                decay_kind=0, beta=None, decay=None, silu=False, run_state=None, run_len=0):
     """The recurrence S_t = diag(a_t) S_{t-1} + k_t v_t^T, o_t = S_t^T q_t (+ skip v_t) per sequence and head over the
     state [slots, heads, n_rows, n_cols] (float32, updated in place).  Give `z` [T, heads * n_rows] for a decay per
     row, a = sigmoid(z + z_bias)^(1 / tau); or `dt` [T, heads] for a decay per head with a step size,
     dt' = softplus(dt + dt_bias), a = exp(-exp(a_log) dt'), v' = dt' v.  All rows float32 (column slices allowed).
     `decay_ready`: `z` already holds a (`row_decay` ran over it).  `q_scale` multiplies the outputs' S^T q.
     `decay_kind` 1 (with `z` and `a_log`): a = exp(-exp(a_log[head]) softplus(z + z_bias)).  `beta` [T, heads]
-    (before its sigmoid, with `z`): the delta rule, after the decay u = sigmoid(beta) (v - S^T k), S += k u^T."""
+    (before its sigmoid, with `z`): the delta rule, after the decay u = sigmoid(beta) (v - S^T k), S += k u^T.
+    `decay` (float32 [heads], instead of `z` and `dt`): one constant factor per head; `silu`: k, q and v pass silu on
+    their way in.  With `run_len` the tokens of every sequence are cut into runs of that many that are scanned side by
+    side; `run_state` float32 [>= sequences * runs, heads, n_rows, n_cols] is scratch, runs = ceil(most new tokens /
+    run_len)."""
+    global launch_count
+    runs = 0
+    if run_len:
+        runs = -(-batch.max_new // run_len)
+        assert run_state.dtype == torch.float32 and run_state.is_contiguous() and run_state.is_cuda
+        assert run_state.numel() >= batch.n_seqs * runs * n_heads * n_rows * n_cols
+    assert decay is None or (decay.is_cuda and decay.dtype == torch.float32 and decay.is_contiguous() and decay.numel() == n_heads)
     small = [t for t in (z_bias, dt_bias, a_log, skip) if t is not None]
     _need_cuda(k, q, v, state, out, z, dt, beta, *small)
     for t in (k, q, v, out, z, dt, beta):
@@ -720,7 +759,16 @@ def linear_scan(k, q, v, state, out, batch, *, n_heads, heads_per_group, n_rows,
           c_float(q_scale), _p(state), _p(out), c_long(out.stride(0)), _p(batch.seq_slot), _p(batch.seq_tok0),
           _p(batch.seq_new), c_int(batch.n_seqs), c_int(getattr(batch, "max_new", 1 << 20)), c_int(n_heads),
           c_int(heads_per_group), c_int(n_rows), c_int(n_cols), c_int(int(decay_ready)), c_int(int(decay_kind)),
-          _p(beta), c_long(0 if beta is None else beta.stride(0)), _stream())
+          _p(beta), c_long(0 if beta is None else beta.stride(0)), _p(decay), c_int(int(silu)), _p(run_state),
+          c_int(int(run_len)), c_int(runs), _stream())
+    launch_count += 2 if run_len else 0
+
+
+def silu_rows(x):
+    """x <- silu(x) in place: float32 rows (a column slice allowed)."""
+    _need_cuda(x)
+    assert x.dtype == torch.float32 and x.dim() == 2 and x.stride(1) == 1
+    _call("cpi_silu_rows", _p(x), c_long(x.stride(0)), c_int(x.shape[0]), c_int(x.shape[1]), _stream())
 
 
 def row_decay(z, z_bias, tau, *, kind=0, a_log=None, rows_per_head=0):

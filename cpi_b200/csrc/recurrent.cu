@@ -15,6 +15,12 @@
 //                      A row decay may also be a_t = exp(-exp(A_log[head]) * softplus(z_t + bias)).  With `beta`
 //                      the update is the delta rule: after the decay, u_t = beta_t (v_t - S^T k_t), S += k_t u_t^T,
 //                      o_t = S^T q_t (the read-out sees the token's own write).
+//                      A third flavour has one constant decay per head, a_t = decay[h]; k, q and v may then pass silu
+//                      on their way in.  Because a run of n tokens multiplies its entry state by decay^n whatever the
+//                      tokens are, a long prompt of this flavour is cut into runs that are scanned side by side: every
+//                      run from a zero state for what it adds (no outputs), the runs' entry states by one pass over
+//                      them (scan_chain), and every run again from its true entry state for the outputs.
+//   silu_rows          rows made silu(row) in place: what a prompt's recurrence would otherwise redo per block of columns.
 //   rglru_scan         a gated linear recurrent unit with one state element per channel (see its own comment);
 //   block_major_rows   the equal parts of float32 rows laid out part by part, as the rows of a grouped product.
 //   head_unit          rows of heads made unit vectors in place: x / sqrt(sum(x^2) + eps) per head.
@@ -105,7 +111,12 @@ struct ScanParams {
   int decay_ready;                       // z already holds the decays a (row_decay ran over it)
   int decay_kind;                        // row flavour: 0 a = sigmoid(z + b)^(1/tau), 1 a = exp(-exp(a_log[head]) softplus(z + b))
   const float* beta; long beta_stride;   // [T, H] before the sigmoid, or null; with it the update is the delta rule
+  const float* decay; int silu;          // constant flavour: [H]; whether k, q and v pass silu here
+  int run_len, runs;                     // constant flavour: > 0: block x takes run x % runs (run_len tokens) of sequence x / runs,
+                                         // and `state` holds an entry per (sequence, run) instead of one per slot
 };
+
+enum ScanDecay : int { kStepDecay = 0, kRowDecay = 1, kConstDecay = 2, kConstDecayRuns = 3 };      // the last: what a run adds, no outputs
 
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.0f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ float log_sigmoid_f(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
@@ -153,16 +164,18 @@ template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile(
 // copied into what the recurrence needs (a = sigmoid(z + b)^(1/tau) unless the caller prepared it, or the step
 // size and the head's decay); q's constant scale multiplies the output sum.  Per token the rows' k, q and a lie as each lane group's NPT values followed by four words of padding,
 // so that the 16-byte reads of different kk fall into different banks.
-template <int NPT, int KS, bool ROW_DECAY, int CPT, bool DELTA>
+template <int NPT, int KS, int DECAY, int CPT, bool DELTA>
 __global__ void __launch_bounds__(256) linear_scan_kernel(ScanParams p) {
   // A decode step (one token staged at a time) lets the kernel behind it start at once.  A prompt does not: its few
   // blocks run for hundreds of microseconds, one to a multiprocessor, on a chain of dependent instructions, and
   // thousands of blocks of the next kernel waiting beside them were measured to slow that chain by half.
   if (p.chunk == 1) pdl_launch_dependents();
   extern __shared__ __align__(16) float smem[];
+  constexpr bool ROW_DECAY = DECAY == kRowDecay, STEP_DECAY = DECAY == kStepDecay, READS = DECAY != kConstDecayRuns;
+  constexpr bool CONST_DECAY = !ROW_DECAY && !STEP_DECAY;
   constexpr int PVW = 32 / KS, ROWP = KS * (NPT + 4), NVEC = ROW_DECAY ? 3 : 2;
   const int nwarps = blockDim.x >> 5, pvb = nwarps * PVW * CPT;
-  const int s = blockIdx.x, h = blockIdx.y;
+  const int s = CONST_DECAY && p.run_len > 0 ? blockIdx.x / p.runs : blockIdx.x, h = blockIdx.y;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, kk = lane / PVW, pp = lane % PVW;
   const int lcol = (warp * PVW + pp) * CPT;                  // this thread's first column within the block's slice
   const int col0 = blockIdx.z * pvb, col = col0 + lcol;
@@ -181,7 +194,8 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(ScanParams p) {
   // (rows past the state's size and columns past the head's are never copied into and stay zero)
   float head_a = 0.f, head_dtb = 0.f, head_skip = 0.f, head_rate = 0.f;
   if (ROW_DECAY && p.decay_kind == 1) head_rate = expf(load_any(p.a_log, p.small_dtype, h));
-  if (!ROW_DECAY) {
+  if (CONST_DECAY) head_a = p.decay[h];
+  if (STEP_DECAY) {
     head_a = -expf(load_any(p.a_log, p.small_dtype, h));
     head_dtb = p.dt_bias ? load_any(p.dt_bias, p.small_dtype, h) : 0.f;
   }
@@ -191,8 +205,16 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(ScanParams p) {
     for (int n = tid; n < KS * NPT; n += blockDim.x)
       bias_s[n] = (n < N && p.z_bias) ? load_any(p.z_bias, p.small_dtype, (size_t)h * N + n) : 0.f;
   pdl_wait();
-  const int n_tok = p.seq_new[s], tok0 = p.seq_tok0[s];
-  float* st = p.state + (((size_t)p.seq_slot[s] * H + h) * N) * Dv + col;
+  int n_tok = p.seq_new[s], tok0 = p.seq_tok0[s];
+  size_t home = p.seq_slot[s];
+  if (CONST_DECAY && p.run_len > 0) {                        // one run of the sequence's tokens
+    const int first = (int)(blockIdx.x % p.runs) * p.run_len;
+    n_tok = min(p.run_len, n_tok - first);
+    if (n_tok <= 0) return;                                  // (the whole block: nobody waits for it)
+    tok0 += first;
+    home = blockIdx.x;
+  }
+  float* st = p.state + ((home * H + h) * N) * Dv + col;
   // rows kk * NPT .., columns col .. col + CPT - 1; two neighbouring rows of a column make one pair, so that the
   // recurrence runs on the packed float32 instructions (each half rounds as the single instruction does)
   float2 S[NPT / 2][CPT];
@@ -201,7 +223,7 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(ScanParams p) {
     const int n = kk * NPT + i;
 #pragma unroll
     for (int c = 0; c < CPT; ++c) {
-      const float s0 = (col + c < Dv && n < N) ? st[(size_t)n * Dv + c] : 0.f;
+      const float s0 = READS && col + c < Dv && n < N ? st[(size_t)n * Dv + c] : 0.f;
       if (i & 1) S[i / 2][c].y = s0; else S[i / 2][c].x = s0;
     }
   }
@@ -218,7 +240,7 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(ScanParams p) {
         const int at = j * ROWP + (n / NPT) * (NPT + 4) + n % NPT;
         const size_t t = (size_t)(tok0 + c0 + j);
         cp_async16(ks + at, p.k + t * p.k_stride + (size_t)g * N + n);
-        cp_async16(qs + at, p.q + t * p.q_stride + (size_t)g * N + n);
+        if (READS) cp_async16(qs + at, p.q + t * p.q_stride + (size_t)g * N + n);
         if (ROW_DECAY) cp_async16(ds + at, p.z + t * p.z_stride + (size_t)h * N + n);
       }
     } else {
@@ -228,7 +250,7 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(ScanParams p) {
         const int at = j * ROWP + (n / NPT) * (NPT + 4) + n % NPT;
         const size_t t = (size_t)(tok0 + c0 + j);
         cp_async4(ks + at, p.k + t * p.k_stride + (size_t)g * N + n);
-        cp_async4(qs + at, p.q + t * p.q_stride + (size_t)g * N + n);
+        if (READS) cp_async4(qs + at, p.q + t * p.q_stride + (size_t)g * N + n);
         if (ROW_DECAY) cp_async4(ds + at, p.z + t * p.z_stride + (size_t)h * N + n);
       }
     }
@@ -237,7 +259,7 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(ScanParams p) {
       const int j = e / pvb, c = col0 + e % pvb;
       if (c < Dv) cp_async4(vs + e, p.v + (size_t)(tok0 + c0 + j) * p.v_stride + (size_t)h * Dv + c);
     }
-    if (!ROW_DECAY) {
+    if (STEP_DECAY) {
       float* dts = dt_of(b);
       for (int j = tid; j < nc; j += blockDim.x) cp_async4(dts + j, p.dt + (size_t)(tok0 + c0 + j) * p.dt_stride + h);
     }
@@ -259,7 +281,16 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(ScanParams p) {
     __syncthreads();
     // what was copied becomes what the recurrence needs
     float *ks = k_of(b), *qs = q_of(b), *ds = d_of(b), *vs = v_of(b), *dts = dt_of(b), *as = a_of(b);
-    const bool transform = ROW_DECAY ? !p.decay_ready : true;
+    const bool transform = ROW_DECAY ? !p.decay_ready : CONST_DECAY ? p.silu != 0 : true;
+    if (CONST_DECAY && transform) {                          // (rows and columns past the sizes are zeros and stay zeros)
+      for (int e = tid; e < nc * ROWP; e += blockDim.x) {
+        const int within = e % (NPT + 4);
+        if (within >= NPT) continue;                         // padding
+        ks[e] = silu_f(ks[e]);
+        if (READS) qs[e] = silu_f(qs[e]);
+      }
+      for (int e = tid; e < nc * pvb; e += blockDim.x) vs[e] = silu_f(vs[e]);
+    }
     if (ROW_DECAY && transform) {
       for (int e = tid; e < nc * KS * NPT; e += blockDim.x) {
         const int j = e / (KS * NPT), n = e % (KS * NPT);
@@ -270,7 +301,7 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(ScanParams p) {
     }
     if (DELTA)
       for (int j = tid; j < nc; j += blockDim.x) dts[j] = 1.0f / (1.0f + expf(-dts[j]));
-    if (!ROW_DECAY) {
+    if (STEP_DECAY) {
       for (int j = tid; j < nc; j += blockDim.x) {
         const float dt = softplus_f(dts[j] + head_dtb);
         dts[j] = dt;
@@ -286,7 +317,8 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(ScanParams p) {
       float v_raw[CPT], o[CPT];
       float2 vv[CPT], o2[CPT];
       float a = 0.f, dtj = 1.f;
-      if (!ROW_DECAY) { dtj = dts[j]; a = as[j]; }
+      if (STEP_DECAY) { dtj = dts[j]; a = as[j]; }
+      if (CONST_DECAY) a = head_a;
 #pragma unroll
       for (int c = 0; c < CPT; ++c) {
         v_raw[c] = vs[j * pvb + lcol + c];
@@ -364,12 +396,12 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(ScanParams p) {
 #pragma unroll
           for (int c = 0; c < CPT; ++c) {
             S[2 * i4 + r][c] = __ffma2_rn(kr[r], vv[c], __fmul2_rn(dr[r], S[2 * i4 + r][c]));
-            o2[c] = __ffma2_rn(S[2 * i4 + r][c], qr[r], o2[c]);
+            if (READS) o2[c] = __ffma2_rn(S[2 * i4 + r][c], qr[r], o2[c]);
           }
         }
       }
       }
-      if constexpr (!DELTA) {                                // (the delta rule has stored its outputs above)
+      if constexpr (!DELTA && READS) {                       // (the delta rule has stored its outputs above)
 #pragma unroll
       for (int c = 0; c < CPT; ++c) {
         o[c] = o2[c].x + o2[c].y;
@@ -383,6 +415,7 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(ScanParams p) {
     __syncthreads();                                         // the buffer may be copied into again
   }
   cp_async_wait<0>();
+  if (DECAY == kConstDecay && p.run_len > 0) return;         // the chain of the runs has left the sequence's state
 #pragma unroll
   for (int i = 0; i < NPT; ++i) {
     const int n = kk * NPT + i;
@@ -444,9 +477,61 @@ __global__ void __launch_bounds__(128) head_unit_kernel(float* x, long stride, i
   for (int i = lane; i < dim; i += 32) r[i] *= inv;
 }
 
-template <int NPT, int KS, bool ROW, int CPT = 1>
+
+// z <- silu(z) over n columns of float32 rows, in place
+__global__ void __launch_bounds__(256) silu_rows_kernel(float* x, long stride, int n, int vec) {
+  // (no early launch of the recurrence behind it: see row_decay_kernel)
+  pdl_wait();
+  float* r = x + (size_t)blockIdx.x * stride;
+  const int i = blockIdx.y * blockDim.x + threadIdx.x;
+  if (vec) {
+    if (4 * i >= n) return;
+    float4 v = reinterpret_cast<float4*>(r)[i];
+    reinterpret_cast<float4*>(r)[i] = make_float4(silu_f(v.x), silu_f(v.y), silu_f(v.z), silu_f(v.w));
+  } else if (i < n) {
+    r[i] = silu_f(r[i]);
+  }
+}
+
+// The runs of the constant flavour, in order: run[r] holds what run r adds and becomes the state it starts from; the
+// sequence's state becomes the one after its last run.
+struct ScanChainParams {
+  float* run;                            // [sequences, runs, H, N Dv]
+  float* state;                          // [slots, H, N Dv]
+  const float* decay;                    // [H]
+  const int* seq_slot; const int* seq_new;
+  int n_heads, run_len, runs; long elems;           // elems = N Dv
+};
+
+__global__ void __launch_bounds__(256) scan_chain_kernel(ScanChainParams p) {
+  pdl_wait();                            // (no early launch of the recurrence behind it: see row_decay_kernel)
+  const long e = (long)blockIdx.z * blockDim.x + threadIdx.x;
+  if (e >= p.elems) return;
+  const int s = blockIdx.x, h = blockIdx.y, n = p.seq_new[s], live = (n + p.run_len - 1) / p.run_len;
+  const float a = p.decay[h], whole = powf(a, (float)p.run_len);
+  float* st = p.state + ((size_t)p.seq_slot[s] * p.n_heads + h) * p.elems + e;
+  float* run = p.run + ((size_t)s * p.runs * p.n_heads + h) * p.elems + e;
+  const size_t step = (size_t)p.n_heads * p.elems;
+  float S = *st;
+  for (int r0 = 0; r0 < live; r0 += 4) {                     // four runs' loads in flight
+    float add[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) add[k] = r0 + k < live ? run[(size_t)(r0 + k) * step] : 0.f;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int r = r0 + k;
+      if (r >= live) break;
+      run[(size_t)r * step] = S;
+      S = fmaf(r == live - 1 ? powf(a, (float)(n - r * p.run_len)) : whole, S, add[k]);
+    }
+  }
+  *st = S;
+}
+
+template <int NPT, int KS, int DECAY, int CPT = 1>
 static int launch_scan(const ScanParams& p0, int n_seqs, int max_new, int max_warps, cudaStream_t stream) {
   ScanParams p = p0;
+  constexpr bool ROW = DECAY == kRowDecay;
   constexpr int PVW = 32 / KS, ROWP = KS * (NPT + 4);
   int nwarps = (p.n_cols + PVW * CPT - 1) / (PVW * CPT);
   if (nwarps > max_warps) nwarps = max_warps;
@@ -461,7 +546,7 @@ static int launch_scan(const ScanParams& p0, int n_seqs, int max_new, int max_wa
   const size_t smem = ((size_t)2 * per_buf + KS * NPT) * sizeof(float);
   auto aligned = [](const float* q, long stride) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0 && stride % 4 == 0; };
   p.vec16 = p.n_rows % 4 == 0 && aligned(p.k, p.k_stride) && aligned(p.q, p.q_stride) && (!ROW || aligned(p.z, p.z_stride));
-  auto kern = ROW && p.beta ? linear_scan_kernel<NPT, KS, ROW, CPT, ROW> : linear_scan_kernel<NPT, KS, ROW, CPT, false>;
+  auto kern = ROW && p.beta ? linear_scan_kernel<NPT, KS, DECAY, CPT, ROW> : linear_scan_kernel<NPT, KS, DECAY, CPT, false>;
   static bool attr_set[2] = {false, false};                  // per instantiation
   if (smem > 48 * 1024 && !attr_set[p.beta != nullptr]) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess) {
@@ -480,7 +565,7 @@ static int launch_scan(const ScanParams& p0, int n_seqs, int max_new, int max_wa
 // lanes share a column, eight warps (16 columns) per block: four times the threads and a quarter of the
 // instructions per thread and token, for a prompt of one or a few sequences, where the token-by-token chain of one
 // (sequence, head) is what the step waits for and most of the GPU would idle.
-template <bool ROW>
+template <int DECAY>
 static int dispatch_scan(const ScanParams& p, int n_seqs, int max_new, cudaStream_t stream) {
   const int N = p.n_rows;
   const long narrow_blocks = (long)n_seqs * p.n_heads * ((p.n_cols + 15) / 16);
@@ -494,21 +579,21 @@ static int dispatch_scan(const ScanParams& p, int n_seqs, int max_new, cudaStrea
     // store -- then weighs more than the rows.  Taking the shuffle sums of four tokens side by side changed
     // nothing: 2.6 ms.  Measured again with prepared decays and paired rows: 4.4 against 2.2 ms; twice the blocks
     // stage and read twice the rows of k, q and the decays.)
-    if (N <= 64) return launch_scan<4, 16, ROW>(p, n_seqs, max_new, 8, stream);
-    if (N <= 128) return launch_scan<8, 16, ROW>(p, n_seqs, max_new, 8, stream);
-    if (N <= 192) return launch_scan<12, 16, ROW>(p, n_seqs, max_new, 8, stream);
-    return launch_scan<16, 16, ROW>(p, n_seqs, max_new, 8, stream);
+    if (N <= 64) return launch_scan<4, 16, DECAY>(p, n_seqs, max_new, 8, stream);
+    if (N <= 128) return launch_scan<8, 16, DECAY>(p, n_seqs, max_new, 8, stream);
+    if (N <= 192) return launch_scan<12, 16, DECAY>(p, n_seqs, max_new, 8, stream);
+    return launch_scan<16, 16, DECAY>(p, n_seqs, max_new, 8, stream);
   }
-  if (N <= 16) return launch_scan<4, 4, ROW>(p, n_seqs, max_new, 2, stream);
-  if (N <= 32) return launch_scan<8, 4, ROW>(p, n_seqs, max_new, 2, stream);
-  if (N <= 48) return launch_scan<12, 4, ROW>(p, n_seqs, max_new, 2, stream);
-  if (N <= 64) return launch_scan<16, 4, ROW>(p, n_seqs, max_new, 2, stream);
-  if (N <= 96) return launch_scan<24, 4, ROW>(p, n_seqs, max_new, 2, stream);
-  if (N <= 128) return launch_scan<32, 4, ROW>(p, n_seqs, max_new, 2, stream);
-  if (N <= 192) return launch_scan<48, 4, ROW>(p, n_seqs, max_new, 2, stream);
-  if (N <= 256) return launch_scan<64, 4, ROW>(p, n_seqs, max_new, 2, stream);
-  if (N <= 512) return launch_scan<64, 8, ROW>(p, n_seqs, max_new, 2, stream);
-  if (N <= 1024) return launch_scan<64, 16, ROW>(p, n_seqs, max_new, 2, stream);
+  if (N <= 16) return launch_scan<4, 4, DECAY>(p, n_seqs, max_new, 2, stream);
+  if (N <= 32) return launch_scan<8, 4, DECAY>(p, n_seqs, max_new, 2, stream);
+  if (N <= 48) return launch_scan<12, 4, DECAY>(p, n_seqs, max_new, 2, stream);
+  if (N <= 64) return launch_scan<16, 4, DECAY>(p, n_seqs, max_new, 2, stream);
+  if (N <= 96) return launch_scan<24, 4, DECAY>(p, n_seqs, max_new, 2, stream);
+  if (N <= 128) return launch_scan<32, 4, DECAY>(p, n_seqs, max_new, 2, stream);
+  if (N <= 192) return launch_scan<48, 4, DECAY>(p, n_seqs, max_new, 2, stream);
+  if (N <= 256) return launch_scan<64, 4, DECAY>(p, n_seqs, max_new, 2, stream);
+  if (N <= 512) return launch_scan<64, 8, DECAY>(p, n_seqs, max_new, 2, stream);
+  if (N <= 1024) return launch_scan<64, 16, DECAY>(p, n_seqs, max_new, 2, stream);
   set_error("linear_scan: a state of %d rows per head is not supported (up to 1024)", N);
   return 1;
 }
@@ -682,9 +767,14 @@ extern "C" int cpi_linear_scan(const float* k, long k_stride, const float* q, lo
                                long out_stride, const int* seq_slot, const int* seq_tok0, const int* seq_new,
                                int n_seqs, int max_new, int n_heads, int heads_per_group, int n_rows, int n_cols,
                                int decay_ready, int decay_kind, const float* beta, long beta_stride,
+                               const float* decay, int silu, float* run_state, int run_len, int runs,
                                cudaStream_t stream) {
   if (n_seqs == 0) return 0;
-  CPI_REQUIRE((z != nullptr) != (dt != nullptr), "linear_scan: give row decays or step sizes, one of the two");
+  CPI_REQUIRE((z != nullptr) + (dt != nullptr) + (decay != nullptr) == 1,
+              "linear_scan: give row decays, step sizes or constant decays, one of the three");
+  CPI_REQUIRE(run_len == 0 || (decay != nullptr && run_state != nullptr && run_len > 0 && runs > 0 &&
+                               (long)run_len * runs >= max_new && (long)n_seqs * runs <= 0x7fffffffL),
+              "linear_scan: %d runs of %d tokens go with constant decays and cover the step", runs, run_len);
   CPI_REQUIRE(dt == nullptr || a_log != nullptr, "linear_scan: step sizes need the heads' decay rates");
   CPI_REQUIRE(n_heads > 0 && heads_per_group > 0 && n_heads % heads_per_group == 0 && n_rows > 0 && n_cols > 0,
               "linear_scan: bad sizes heads=%d per group=%d rows=%d columns=%d", n_heads, heads_per_group, n_rows, n_cols);
@@ -694,9 +784,29 @@ extern "C" int cpi_linear_scan(const float* k, long k_stride, const float* q, lo
   CPI_REQUIRE(beta == nullptr || z != nullptr, "linear_scan: the delta rule comes with row decays");
   ScanParams p{k, k_stride, q, q_stride, v, v_stride, z, z_stride, z_bias, inv_tau, dt, dt_stride, dt_bias, a_log,
                skip, small_dtype, q_scale, state, out, out_stride, seq_slot, seq_tok0, seq_new,
-               n_heads, heads_per_group, n_rows, n_cols, 0, 0, decay_ready, decay_kind, beta, beta_stride};
+               n_heads, heads_per_group, n_rows, n_cols, 0, 0, decay_ready, decay_kind, beta, beta_stride,
+               decay, silu, 0, 1};
   if (max_new < 1) max_new = 1;
-  return z ? dispatch_scan<true>(p, n_seqs, max_new, stream) : dispatch_scan<false>(p, n_seqs, max_new, stream);
+  if (decay) {
+    if (run_len == 0) return dispatch_scan<kConstDecay>(p, n_seqs, max_new, stream);
+    p.state = run_state; p.run_len = run_len; p.runs = runs;
+    if (int rc = dispatch_scan<kConstDecayRuns>(p, n_seqs * runs, run_len, stream)) return rc;
+    ScanChainParams c{run_state, state, decay, seq_slot, seq_new, n_heads, run_len, runs, (long)n_rows * n_cols};
+    const long z_blocks = (c.elems + 255) / 256;
+    CPI_REQUIRE(z_blocks <= 65535, "linear_scan: a state of %d x %d", n_rows, n_cols);
+    cpi::launch_pdl(scan_chain_kernel, dim3(n_seqs, n_heads, (unsigned)z_blocks), dim3(256), 0, stream, c);
+    if (int rc = check_launch("scan_chain")) return rc;
+    return dispatch_scan<kConstDecay>(p, n_seqs * runs, run_len, stream);
+  }
+  return z ? dispatch_scan<kRowDecay>(p, n_seqs, max_new, stream) : dispatch_scan<kStepDecay>(p, n_seqs, max_new, stream);
+}
+
+extern "C" int cpi_silu_rows(float* x, long stride, int n_rows, int n, cudaStream_t stream) {
+  if (n_rows == 0 || n == 0) return 0;
+  const int vec = (reinterpret_cast<uintptr_t>(x) & 15) == 0 && stride % 4 == 0 && n % 4 == 0;
+  const int items = vec ? n / 4 : n;
+  cpi::launch_pdl(silu_rows_kernel, dim3(n_rows, (items + 255) / 256), dim3(256), 0, stream, x, stride, n, vec);
+  return check_launch("silu_rows");
 }
 
 extern "C" int cpi_row_decay(float* z, long z_stride, const void* bias, int bias_dtype, float inv_tau, int n_tokens,

@@ -5,3 +5,4 @@ from . import savenex  # noqa: F401
 from . import nogapel  # noqa: F401
 from . import kikerax  # noqa: F401
 from . import nekorax  # noqa: F401
+from . import delilorn  # noqa: F401

@@ -46,7 +46,8 @@ j * base^(-2m / value_dim) in the position part's layout of pairs, and cached so
 back by i), `output_gate` "elementwise" (tensor "g" [heads * value_dim, hidden]: the concatenated heads are multiplied by
 sigmoid(g h) element by element; True is the gate per head above), and `sink` {"constant": c} (every head's sink has the
 score c and no tensor: 0 adds one to the softmax denominators).  A mixer without biases, norms, value mixing and
-temperature does its convolution, rotations and cache write in one kernel (`qkv_conv_rotate`) when its sizes allow it.
+temperature does its convolution (if any), rotations and cache write in one kernel (`qkv_conv_rotate`) when its sizes
+allow it.
 
 `attend(...)` below is the choice of the attention kernel for prepared queries and a paged cache; other mixers that
 end in softmax attention over pages (`latent_attention`) call it too.
@@ -397,7 +398,7 @@ class AttentionMixer(Mixer):
     def _fused_preparation(self, cache) -> bool:
         return (use_fused_preparation and self.has_kv and cache.owns and self.maps == 1 and not self.bias and not self.qk_norm
                 and self.value_mix is None and not self.values_from_keys and self.temperature is None
-                and (self.taps is not None or self.v_inv_freq is not None) and self.w_qkv.shape[0] % 4 == 0
+                and self.w_qkv.shape[0] % 4 == 0
                 and K.qkv_conv_rotate_supported(self.d, self.dv, self.rot_dims if self.rotary is not None else 0,
                                                 self.v_inv_freq is not None, self.taps or 1))
 

@@ -28,6 +28,10 @@ moe_swiglu    params: hidden_size, num_experts, top_k, expert_size, shared_size 
               tensors: feed_forward.router.weight [E, H], feed_forward.experts.gate_up_proj [E, H, 2I],
               feed_forward.experts.down_proj [E, I, H], feed_forward.shared_expert.{gate,up,down}_proj.weight
 
+moe_mlp       the same with experts that have no gate: down(act(up h)), activation "relu_squared" or "gelu_tanh" as in
+              dense_mlp; expert_names {"up", "down"} in the "per_expert" layout (the only one).  Identity experts, the
+              router's gates and rules, and a shared expert are those of moe_swiglu.
+
 dense_mlp     params: hidden_size, intermediate_size, activation ("relu_squared": max(z, 0)^2, or "gelu_tanh"), tensor_names (up, down):
               down(act(up h)), no gate.  The activation acts on the float32 accumulator of the first product, so its
               input is rounded once, after it.
@@ -116,11 +120,14 @@ class DenseSwiGLU(FeedForward):
             project(a, self.w_down, residual, MODE_ADD if add else MODE_STORE, row_scale=scale)
 
 
+UNGATED_ACTIVATIONS = {"relu_squared": MODE_STORE_RELU2, "gelu_tanh": MODE_STORE_GELU}
+
+
 @register_feed_forward("dense_mlp")
 class DenseMLP(FeedForward):
     graph_safe = True
     can_store = True
-    ACTIVATIONS = {"relu_squared": MODE_STORE_RELU2, "gelu_tanh": MODE_STORE_GELU}
+    ACTIVATIONS = UNGATED_ACTIVATIONS
 
     def __init__(self, spec, prefix="", workspace=None):
         super().__init__(spec, prefix)
@@ -152,6 +159,11 @@ class DenseMLP(FeedForward):
 @register_feed_forward("moe_swiglu")
 class MoESwiGLU(FeedForward):
     graph_safe = True
+    gated = True
+    DEFAULT_ACTIVATION = "silu"
+    # the first product's mode, by activation (the activation is part of its epilogue)
+    ACTIVATIONS = {"silu": MODE_SWIGLU, "gelu_tanh": MODE_GEGLU, "swish_clamped": MODE_CLAMPED_GLU}
+
     def __init__(self, spec, prefix="", workspace=None):
         super().__init__(spec, prefix)
         p = spec.params
@@ -160,9 +172,9 @@ class MoESwiGLU(FeedForward):
         self.gate_mode = p.get("router_gate", "sigmoid_input")
         if self.gate_mode not in ("sigmoid_input", "sigmoid_output", "none", "softmax_chosen", "sigmoid_normed", "scored"):
             raise ValueError(f"moe_swiglu: unknown router_gate '{self.gate_mode}'")
-        self.activation, self.limit = p.get("activation", "silu"), float(p.get("limit") or 0.0)
-        if self.activation not in K.GATE_ACTS:
-            raise ValueError(f"moe_swiglu: unknown activation '{self.activation}'; known: {sorted(K.GATE_ACTS)}")
+        self.activation, self.limit = p.get("activation", self.DEFAULT_ACTIVATION), float(p.get("limit") or 0.0)
+        if self.activation not in self.ACTIVATIONS:
+            raise ValueError(f"{spec.kind}: unknown activation '{self.activation}'; known: {sorted(self.ACTIVATIONS)}")
         if self.activation == "swish_clamped" and not self.limit > 0:
             raise ValueError("moe_swiglu: the clamped activation needs a positive limit")
         self.n_identity = int(p.get("identity_experts") or 0)
@@ -203,8 +215,12 @@ class MoESwiGLU(FeedForward):
         if self.layout not in ("stacked", "per_expert"):
             raise ValueError(f"moe_swiglu: unknown expert_layout '{self.layout}'")
         self.expert_names = {k: prefix + v for k, v in (p.get("expert_names") or {}).items()}
-        if self.layout == "per_expert" and set(self.expert_names) != {"gate", "up", "down"}:
-            raise ValueError("moe_swiglu: the per_expert layout needs expert_names for gate, up and down")
+        # what the first product reads, stacked into one matrix per expert
+        self.inputs = ("gate", "up") if self.gated else ("up",)
+        if self.layout == "per_expert" and set(self.expert_names) != {*self.inputs, "down"}:
+            raise ValueError(f"{spec.kind}: the per_expert layout needs expert_names for {', '.join(self.inputs)} and down")
+        if self.layout == "stacked" and not self.gated:
+            raise ValueError(f"{spec.kind}: experts without a gate are stored one by one (expert_layout 'per_expert')")
         self.b_router = None
         self.shared = None
         if p.get("shared") is not None:
@@ -237,9 +253,8 @@ class MoESwiGLU(FeedForward):
             reqs.append(TensorReq(self.n_choice_bias, (self.n_routed,)))
         if self.layout == "per_expert":
             for e in range(self.n_experts):
-                reqs += [TensorReq(self.expert_names["gate"].format(e=e), (self.inter, self.hidden)),
-                         TensorReq(self.expert_names["up"].format(e=e), (self.inter, self.hidden)),
-                         TensorReq(self.expert_names["down"].format(e=e), (self.hidden, self.inter))]
+                reqs += [TensorReq(self.expert_names[n].format(e=e), (self.inter, self.hidden)) for n in self.inputs]
+                reqs.append(TensorReq(self.expert_names["down"].format(e=e), (self.hidden, self.inter)))
         else:
             reqs += [TensorReq(self.n_gate_up, (self.n_experts, self.hidden, 2 * self.inter)),
                      TensorReq(self.n_down, (self.n_experts, self.inter, self.hidden))]
@@ -255,8 +270,9 @@ class MoESwiGLU(FeedForward):
             self.rule["choice_bias"] = source.get(self.n_choice_bias, device).to(torch.float32).contiguous()
         if self.layout == "per_expert":                                       # stored [out, in] already
             n = self.expert_names
-            self.w_gate_up = torch.stack([_stack(source.get(n["gate"].format(e=e), device), source.get(n["up"].format(e=e), device))
-                                          for e in range(self.n_experts)]).contiguous()             # [E, 2I, H]
+            get = lambda name, e: source.get(n[name].format(e=e), device)
+            self.w_gate_up = torch.stack([_stack(get("gate", e), get("up", e)) if self.gated else get("up", e)
+                                          for e in range(self.n_experts)]).contiguous()             # [E, 2I (or I), H]
             self.w_down = torch.stack([source.get(n["down"].format(e=e), device)
                                        for e in range(self.n_experts)]).contiguous()                # [E, H, I]
         else:
@@ -308,7 +324,7 @@ class MoESwiGLU(FeedForward):
         # identity experts come after the others, so their rows are the last ones and lie outside the products' E groups
         hint = max(1, -(-M // R))
         offsets = offsets[:E + 1]
-        act_mode = {"silu": MODE_SWIGLU, "gelu_tanh": MODE_GEGLU, "swish_clamped": MODE_CLAMPED_GLU}[self.activation]
+        act_mode = self.ACTIVATIONS[self.activation]
         act = ws.get("moe_act", (M, self.inter), h.dtype)
         in_scale = row_scale if self.gate_mode == "sigmoid_input" else None
         with phase("moe_expert"):
@@ -352,3 +368,11 @@ class MoESwiGLU(FeedForward):
             return
         if self.shared is not None:
             self.shared.forward(h, residual, batch)
+
+
+@register_feed_forward("moe_mlp")
+class MoEMLP(MoESwiGLU):
+    """Routed experts of two matrices: the first product's epilogue applies the activation to its float32 sums."""
+    gated = False
+    DEFAULT_ACTIVATION = "relu_squared"
+    ACTIVATIONS = UNGATED_ACTIVATIONS

@@ -10,8 +10,12 @@
                      norm_eps, position (PartSpec; a rotation of rot_dim elements, or "none"; its amplitude multiplies the
                      sines and cosines of both rotated parts), sink (bool), window (None, {"kind": "full"} or {"kind":
                      "sliding", "size": n}: a position sees itself and the n - 1 before it),
-                     tensor_names {"dq", "dq_norm", "uq", "dkv", "dkv_norm", "uk", "uv", "o", "sink"}.
-                     cache: one stream "latent" of one head of kv_rank + rot_dim elements per position.
+                     output_gate (bool; tensor "g" [heads * value_dim, hidden]: the concatenated heads are multiplied by
+                     sigmoid(g h) element by element),
+                     tensor_names {"dq", "dq_norm", "uq", "dkv", "dkv_norm", "uk", "uv", "o", "sink", "g"}.
+                     cache: one stream "latent" of one head of kv_rank + rot_dim elements per position.  A layer that only
+                     runs on another run entry's cache has no dkv and dkv_norm: it reads that entry's latents and rotated
+                     key parts with its own queries, W_uk and W_uv (their kv_rank, rot_dim and rotation are the same).
 
 How it runs.  Only [c | r] is cached, and the keys and values of the heads are never formed: since
 q_n . (W_uk,n c) = (W_uk,n^T q_n) . c, the plain part of a query is first taken through W_uk,n^T (a grouped product, one
@@ -47,13 +51,13 @@ class LatentAttentionMixer(Mixer):
     def __init__(self, spec, prefix="", workspace=None, owns_cache=True):
         super().__init__(spec, prefix)
         p = spec.params
-        if not owns_cache:
-            raise ValueError("latent_attention: reading another run entry's cache is not supported")
+        self.has_kv = bool(owns_cache)                # False: every run entry of this layer reads another's cache
         self.hidden, self.nh = int(p["hidden_size"]), int(p["heads"])
         self.d, self.r, self.dv = int(p["head_dim"]), int(p["rot_dim"]), int(p["value_dim"])
         self.q_rank, self.kv_rank = int(p["q_rank"]), int(p["kv_rank"])
         self.scale, self.eps = float(p["softmax_scale"]), float(p["norm_eps"])
         self.has_sink = bool(p.get("sink", False))
+        self.gate_rows = self.nh * self.dv if p.get("output_gate", False) else 0
         w = p.get("window") or {"kind": "full"}
         if w["kind"] not in ("full", "sliding"):
             raise ValueError(f"latent_attention: a window of kind '{w['kind']}' (full or sliding)")
@@ -70,7 +74,8 @@ class LatentAttentionMixer(Mixer):
         self.position = build_part("position", p["position"])
         tn = {"dq": "mixer.q_a_proj.weight", "dq_norm": "mixer.q_a_norm.weight", "uq": "mixer.q_b_proj.weight",
               "dkv": "mixer.kv_a_proj.weight", "dkv_norm": "mixer.kv_a_norm.weight", "uk": "mixer.k_b_proj.weight",
-              "uv": "mixer.v_b_proj.weight", "o": "mixer.o_proj.weight", "sink": "mixer.sinks"}
+              "uv": "mixer.v_b_proj.weight", "o": "mixer.o_proj.weight", "sink": "mixer.sinks",
+              "g": "mixer.g_proj.weight"}
         tn.update(p.get("tensor_names") or {})
         self.tn = {k: prefix + v for k, v in tn.items()}
         self.ws = workspace
@@ -81,9 +86,12 @@ class LatentAttentionMixer(Mixer):
         t, H = self.tn, self.hidden
         reqs = [TensorReq(t["dq"], (self.q_rank, H)), TensorReq(t["dq_norm"], (self.q_rank,), init="ones+normal"),
                 TensorReq(t["uq"], (self.nh * (self.d + self.r), self.q_rank)),
-                TensorReq(t["dkv"], (self.row, H)), TensorReq(t["dkv_norm"], (self.kv_rank,), init="ones+normal"),
                 TensorReq(t["uk"], (self.nh * self.d, self.kv_rank)), TensorReq(t["uv"], (self.nh * self.dv, self.kv_rank)),
                 TensorReq(t["o"], (H, self.nh * self.dv))]
+        if self.has_kv:
+            reqs += [TensorReq(t["dkv"], (self.row, H)), TensorReq(t["dkv_norm"], (self.kv_rank,), init="ones+normal")]
+        if self.gate_rows:
+            reqs.append(TensorReq(t["g"], (self.gate_rows, H)))
         if self.has_sink:
             reqs.append(TensorReq(t["sink"], (self.nh,)))
         return reqs
@@ -91,15 +99,18 @@ class LatentAttentionMixer(Mixer):
     def load(self, source, device):
         t = self.tn
         f32 = lambda name: source.get(t[name], device).to(torch.float32).contiguous()
-        dq, dkv = source.get(t["dq"], device), source.get(t["dkv"], device)
-        dt = torch.float32 if torch.float32 in (dq.dtype, dkv.dtype) else torch.bfloat16
-        self.w_down = torch.cat([dq.to(dt), dkv.to(dt)], dim=0).contiguous()          # [q_rank + kv_rank + rot, H]
+        # one product for all that reads the layer's input: [gate | query latent | latent and rotated key part]
+        parts = [source.get(t[n], device) for n, on in (("g", self.gate_rows), ("dq", True), ("dkv", self.has_kv)) if on]
+        dt = torch.float32 if any(w.dtype == torch.float32 for w in parts) else torch.bfloat16
+        self.w_down = torch.cat([w.to(dt) for w in parts], dim=0).contiguous()
         self.w_uq = source.get(t["uq"], device).contiguous()
         uk = source.get(t["uk"], device).view(self.nh, self.d, self.kv_rank)
         self.w_ukT = uk.transpose(1, 2).contiguous()                                   # [heads, kv_rank, dim]
         self.w_uv = source.get(t["uv"], device).view(self.nh, self.dv, self.kv_rank).contiguous()
         self.w_o = source.get(t["o"], device).contiguous()
-        self.w_qnorm, self.w_cnorm = f32("dq_norm"), f32("dkv_norm")
+        self.w_qnorm = f32("dq_norm")
+        if self.has_kv:
+            self.w_cnorm = f32("dkv_norm")
         if self.has_sink:
             self.sink = f32("sink")
         self.position.prepare(device)
@@ -122,15 +133,17 @@ class LatentAttentionMixer(Mixer):
         inv_freq = None if self.rotary is None else self.rotary.inv_freq
         inter = self.rotary is not None and self.rotary.interleaved
         amp = 1.0 if self.rotary is None else self.rotary.amplitude
-        down = self.ws.get("latent_down", (T, self.q_rank + row), f32)
+        down = self.ws.get("latent_down", (T, self.w_down.shape[0]), f32)
+        gate, low = down[:, :self.gate_rows], down[:, self.gate_rows:]
         with phase("qkv"):
             project(h, self.w_down, down)
-        with phase("kv_store"):          # the normed latent and the rotated key part of every token go into its page
-            K.latent_kv_write(down[:, self.q_rank:], self.w_cnorm, self.eps, inv_freq, inter, pages, table, page_size,
-                              batch.token_seq, batch.token_pos, batch.seq_slot, rank=rank, rot=R, amplitude=amp)
+        if self.has_kv and cache.owns:
+            with phase("kv_store"):      # the normed latent and the rotated key part of every token go into its page
+                K.latent_kv_write(low[:, self.q_rank:], self.w_cnorm, self.eps, inv_freq, inter, pages, table, page_size,
+                                  batch.token_seq, batch.token_pos, batch.seq_slot, rank=rank, rot=R, amplitude=amp)
         cq = self.ws.get("latent_cq", (T, self.q_rank), dt)
         with phase("rmsnorm"):
-            K.rmsnorm(down[:, :self.q_rank], self.w_qnorm, self.eps, cq)
+            K.rmsnorm(low[:, :self.q_rank], self.w_qnorm, self.eps, cq)
         q = self.ws.get("latent_q", (T, H * (D + R)), f32)
         with phase("qkv"):
             project(cq, self.w_uq, q)
@@ -172,4 +185,8 @@ class LatentAttentionMixer(Mixer):
         with phase("wo"):
             project(lat, self.w_uv, out.view(T * H, self.dv), MODE_STORE, out_rows=rows, group_offsets=offsets,
                     n_groups=H, rows_per_group_hint=T)
+        if self.gate_rows:
+            with phase("head_post"):
+                K.head_turn(out, out, batch.token_pos, n_heads=H, value_dim=self.dv, gate=gate)
+        with phase("wo"):
             project(out, self.w_o, residual, MODE_ADD if add else MODE_STORE)

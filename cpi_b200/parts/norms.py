@@ -48,12 +48,16 @@ class RMSNorm(Norm):
         return out
 
     def enter(self, y, x, following=None, h_out=None):
-        if self.weight_offset:
-            raise ValueError("rmsnorm: a weight stored as a distance from a constant does not norm a sublayer's output here")
-        if isinstance(y, ExpertSum):
-            y = y.rows(self.ws)
-        K.sum_norm_add([y], [1.0], self.weight, x, eps=self.eps, add=True)
-        if following is not None:
+        together = isinstance(following, RMSNorm) and following.weight is not None
+        if self.weight is not None:            # both norms, the sum and the combination of experts: one kernel
+            kw = {"experts": y.lists()} if isinstance(y, ExpertSum) else {"y": y}
+            K.rms_step(x, post=(self.weight, self.weight_offset, self.eps), h_out=h_out if together else None,
+                       pre=(following.weight, following.weight_offset, following.eps) if together else None, **kw)
+        else:
+            together = False
+            y = y.rows(self.ws) if isinstance(y, ExpertSum) else y
+            K.sum_norm_add([y], [1.0], None, x, eps=self.eps, add=True)
+        if following is not None and not together:
             following(x, h_out.dtype, out=h_out)
 
 

@@ -21,7 +21,8 @@ in both precisions; the projections feed them as float32 rows.
           tensor_names {"q", "k", "v", "g", "o", "norm", "a1", "a2", "a2_bias"}.
           state: "s" [heads, key_dim, value_dim].
 
-"rglru" keeps a vector instead of a matrix: one state element per channel, see `RGLRUMixer`.
+"lightning" has one constant decay per head, see `LightningMixer`; "rglru" keeps a vector instead of a matrix: one
+state element per channel, see `RGLRUMixer`.
 """
 from __future__ import annotations
 
@@ -36,6 +37,10 @@ from .linear import MODE_ADD, MODE_STORE, project
 
 # steps whose longest portion has more tokens than this prepare the row decays with a kernel of their own
 DECAY_PREPASS_FROM = 16
+# a recurrence with constant decays is cut into runs of at least this many tokens, until its blocks fill the GPU this often
+RUN_TOKENS = 64
+RUN_BLOCKS_PER_SM = 4
+MAX_STATE_ROWS = 1024             # rows of a head's state that the recurrence's kernel takes
 
 
 def _cat_rows(tensors):
@@ -279,6 +284,92 @@ class GatedDeltaMixer(Mixer):
         with phase("gated_norm"):
             g = self.ws.get("gdr_gated", (T, nv), h.dtype)
             K.gated_norm(o, gate, self.w_norm, g, parts=self.nh, gate_first=False, eps=self.eps, gate_act="sigmoid")
+        with phase("wo"):
+            project(g, self.w_o, residual, MODE_ADD if add else MODE_STORE)
+
+
+@register_mixer("lightning")
+class LightningMixer(Mixer):
+    """Linear attention with one constant decay per head:
+
+        q = silu(W_q h), k = silu(W_k h) (heads of key_dim), v = silu(W_v h) (heads of value_dim);
+        S <- decay[head] S + k v^T;  o = S^T q   (no scale);
+        out = W_o (rmsnorm(all heads' o side by side) * norm * sigmoid(W_g h)).
+
+    params: hidden_size, heads, key_dim, value_dim, decay (a number per head), norm_eps,
+    tensor_names {"q", "k", "v", "g", "o", "norm"}.
+    state: "s" [heads, key_dim, value_dim] float32.  The projections feed the recurrence as float32 rows.
+
+    A decode step's recurrence applies silu itself; a prompt's rows pass it once beforehand.  A long prompt of few
+    sequences is cut into runs that are scanned side by side (`csrc/recurrent.cu`: the runs of `linear_scan`)."""
+    graph_safe = True
+    can_store = True
+
+    def __init__(self, spec, prefix="", workspace=None, owns_cache=True):
+        super().__init__(spec, prefix)
+        p = spec.params
+        self.hidden, self.nh = int(p["hidden_size"]), int(p["heads"])
+        self.dk, self.dv, self.eps = int(p["key_dim"]), int(p["value_dim"]), float(p["norm_eps"])
+        self.decay_values = [float(a) for a in p["decay"]]
+        if len(self.decay_values) != self.nh:
+            raise ValueError(f"lightning: {len(self.decay_values)} decays for {self.nh} heads")
+        if not all(0.0 <= a <= 1.0 for a in self.decay_values):
+            raise ValueError("lightning: a decay is a factor from 0 to 1")
+        if self.dk > MAX_STATE_ROWS:
+            raise ValueError(f"lightning: keys of {self.dk} elements (up to {MAX_STATE_ROWS})")
+        if not owns_cache:
+            raise ValueError("lightning: a recurrent layer cannot read another run entry's state")
+        tn = {"q": "mixer.q_proj.weight", "k": "mixer.k_proj.weight", "v": "mixer.v_proj.weight",
+              "g": "mixer.g_proj.weight", "o": "mixer.o_proj.weight", "norm": "mixer.g_norm.weight"}
+        tn.update(p.get("tensor_names") or {})
+        self.tn = {k: prefix + v for k, v in tn.items()}
+        self.ws = workspace
+        self.w_in = self.w_norm = self.w_o = self.decay = None
+
+    def requirements(self):
+        t, H, nk, nv = self.tn, self.hidden, self.nh * self.dk, self.nh * self.dv
+        return [TensorReq(t["q"], (nk, H)), TensorReq(t["k"], (nk, H)), TensorReq(t["v"], (nv, H)),
+                TensorReq(t["g"], (nv, H)), TensorReq(t["o"], (H, nv)), TensorReq(t["norm"], (nv,), init="ones+normal")]
+
+    def load(self, source, device):
+        t = self.tn
+        self.w_in = _cat_rows([source.get(t[n], device) for n in ("q", "k", "v", "g")])
+        self.w_norm = source.get(t["norm"], device).to(torch.float32).contiguous()
+        self.w_o = source.get(t["o"], device).contiguous()
+        self.decay = torch.tensor(self.decay_values, dtype=torch.float32, device=device)
+
+    def state_requirements(self):
+        return [StateRequirement("s", (self.nh, self.dk, self.dv))]
+
+    def run_length(self, n_seqs: int, max_new: int) -> int:
+        """Tokens of the runs that a step's sequences are cut into, or 0: enough runs to fill the GPU with blocks of the
+        recurrence (one per sequence, run, head and 16 columns), none shorter than RUN_TOKENS."""
+        blocks = n_seqs * self.nh * -(-self.dv // 16)
+        runs = min(-(-RUN_BLOCKS_PER_SM * K.sm_count() // blocks), max_new // RUN_TOKENS)
+        return 0 if runs < 2 else -(-max_new // runs)
+
+    def forward(self, h, residual, batch, cache, add=True):
+        T, f32 = h.shape[0], torch.float32
+        nk, nv = self.nh * self.dk, self.nh * self.dv
+        proj = self.ws.get("lightning_proj", (T, 2 * nk + 2 * nv), f32)           # [q | k | v | g]
+        with phase("qkv"):
+            project(h, self.w_in, proj)
+        o = self.ws.get("lightning_o", (T, nv), f32)
+        with phase("scan"):
+            ready = batch.max_new > DECAY_PREPASS_FROM
+            if ready:
+                K.silu_rows(proj[:, :2 * nk + nv])
+            run_len, run_state = self.run_length(batch.n_seqs, batch.max_new), None
+            if run_len:
+                runs = -(-batch.max_new // run_len)
+                run_state = self.ws.get("lightning_runs", (batch.n_seqs * runs, nv * self.dk), f32)
+            K.linear_scan(proj[:, nk:2 * nk], proj[:, :nk], proj[:, 2 * nk:2 * nk + nv], cache.state("s"), o, batch,
+                          n_heads=self.nh, heads_per_group=1, n_rows=self.dk, n_cols=self.dv, decay=self.decay,
+                          silu=not ready, run_state=run_state, run_len=run_len)
+        with phase("gated_norm"):
+            g = self.ws.get("lightning_gated", (T, nv), h.dtype)
+            K.gated_norm(o, proj[:, 2 * nk + nv:], self.w_norm, g, parts=1, gate_first=False, eps=self.eps,
+                         gate_act="sigmoid")
         with phase("wo"):
             project(g, self.w_o, residual, MODE_ADD if add else MODE_STORE)
 
