@@ -52,6 +52,10 @@ gated delta rule, dense and routed feed-forwards) at the same sizes, measured th
 elementwise gate alternating with windowed attention over a cached latent; tanh norms before and after every sublayer;
 clamped and identity experts chosen from the best groups; a pass entered through a matrix) at two layer sizes beside
 Nogapel's layers (mixers) and Kikerax's (experts, norms on the outputs) at the same sizes, measured the same way.
+`--workload delilorn`: the Delilorn design (attention over a cached latent, linear attention with constant decays,
+attention over the first one's latent, windowed attention with kept first tokens; RMS norms before and after every
+sublayer; ungated experts) at two layer sizes beside Nekorax's layers (latent attention, norms on both sides, experts) and
+Veredra's (gated linear attention, windowed attention) at the same sizes, measured the same way.
 """
 from __future__ import annotations
 
@@ -1259,6 +1263,147 @@ def run_nekorax(args) -> dict:
     return out
 
 
+DELILORN_SIZES = {
+    # width, attention (heads, kv heads, head size, window, kept first tokens), lightning (heads, key size, value size),
+    # latent (heads, plain, rotated, value, query rank, latent rank), experts (count, top, ff): two points with the layer
+    # shapes of 1-3 B and 7-8 B parameter models
+    "w2048": dict(width=2048, attn=(16, 4, 128, 1024, 64), linear=(16, 128, 128), latent=(16, 128, 64, 128, 768, 512), moe=(16, 4, 1536)),
+    "w4096": dict(width=4096, attn=(32, 8, 128, 2048, 64), linear=(32, 128, 128), latent=(32, 128, 64, 128, 1536, 512), moe=(16, 4, 3072)),
+}
+
+
+def delilorn_config(sz: dict, vocab: int, reps: int) -> dict:
+    """(latent attention, lightning, latent attention over the first one's latent, attention) x reps, routed experts."""
+    H, G, D, win, keep = sz["attn"]
+    nh, nk, nv = sz["linear"]
+    lh, ld, lr, lv, qr, kr = sz["latent"]
+    E, top, eff = sz["moe"]
+    mlp = {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": E, "top": top}}
+    latent = {"heads": lh, "dim": ld, "rot_dim": lr, "vdim": lv, "q_rank": qr, "kv_rank": kr, "scale": (ld + lr) ** -0.5,
+              "rot": {"base": 1e4, "dims": lr}}
+    layers = []
+    for r in range(reps):
+        layers += [{"type": "latent_attention", "mixer": latent},
+                   {"type": "lightning", "mixer": {"heads": nh, "dim": nk, "vdim": nv,
+                                                   "decay": [1.0 - 2.0 ** -(2.0 + 8.0 * i / nh) for i in range(nh)]}},
+                   {"type": "latent_attention", "mixer": {**latent, "kv_from": 4 * r}},
+                   {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5,
+                                                   "rot": {"base": 1e6, "dims": D // 2}, "mask": {"size": win, "keep_first": keep}}}]
+    return {"architecture": "Delilorn", "layers": [{**l, "mlp": mlp} for l in layers], "norm": {"eps": 1e-6}, "vocab": vocab,
+            "width": sz["width"]}
+
+
+def nekorax_like_delilorn_config(sz: dict, vocab: int, layers: int) -> dict:
+    """The closest model the library had for latent attention, norms on both sides of a sublayer and routed experts:
+    Nekorax layers of latent attention over everything, without identity experts."""
+    lh, ld, lr, lv, qr, kr = sz["latent"]
+    E, top, eff = sz["moe"]
+    one = {"type": "latent_attention",
+           "mlp": {"kind": "moe", "expert": {"ff": eff, "limit": 7.0}, "router": {"experts": E, "top": top}},
+           "mixer": {"heads": lh, "dim": ld, "rot_dim": lr, "vdim": lv, "q_rank": qr, "kv_rank": kr, "scale": (ld + lr) ** -0.5,
+                     "rot": {"base": 1e4, "dims": lr}}}
+    return {"architecture": "Nekorax", "layers": [one] * layers, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "vocab": vocab,
+            "width": sz["width"]}
+
+
+def veredra_like_delilorn_config(sz: dict, vocab: int, pairs: int) -> dict:
+    """The closest model the library had for linear attention and for windowed attention: Veredra's gated linear attention
+    and its attention at the same head counts and sizes; a small dense feed-forward."""
+    H, G, D, win, _ = sz["attn"]
+    nh, nk, nv = sz["linear"]
+    mlp = {"kind": "dense", "ff": sz["width"]}
+    pair = [{"type": "gla", "mixer": {"heads": nh, "dim": nk, "vdim": nv, "tau": 16.0}, "mlp": mlp},
+            {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5,
+                                            "rot": {"base": 1e6, "dims": D // 2}, "mask": {"size": win}}, "mlp": mlp}]
+    return {"architecture": "Veredra", "layers": pair * pairs, "norm": {"eps": 1e-6}, "streams": 1, "vocab": vocab, "width": sz["width"],
+            "logit_scale": 1.0, "logit_softcap": 30.0}
+
+
+def run_delilorn(args) -> dict:
+    """Prefill and decode of Delilorn at two layer sizes, with the time of every phase per layer that has it and each
+    phase's share of its roofline, beside the like phases of Nekorax layers (latent attention, norms, experts) and Veredra
+    layers (recurrence, windowed attention) at equal sizes: products by flops over the measured bf16 rate in prefill and by
+    weight bytes over the measured copy rate in decode; attention by flops / cache bytes; recurrences and row kernels by
+    bytes (the recurrence's by the state in decode)."""
+    import torch
+
+    pk = peaks()
+    vocab, T, B, reps = 32000, 2048, 8, 1
+    n_layers = 4 * reps
+    g = torch.Generator().manual_seed(7)
+    toks = lambda n: torch.randint(0, vocab, (n,), generator=g).tolist()
+    out = {"metric": "tokens/s, Delilorn beside Nekorax and Veredra layers at equal layer sizes (bf16, random weights)",
+           "unit": "tokens/s", "dtype": "bf16", "data": "synthetic", "peaks": pk, "points": {}}
+    tf, bw = pk["bf16_tflops"] * 1e12, pk["hbm_gbs"] * 1e9
+    sizes = {k: v for k, v in DELILORN_SIZES.items() if not args.sizes or k in args.sizes.split(",")}
+    for name, sz in sizes.items():
+        W = sz["width"]
+        H, G, D, win, keep = sz["attn"]
+        nh, nk, nv = sz["linear"]
+        lh, ld, lr, lv, qr, kr = sz["latent"]
+        E, top, eff = sz["moe"]
+        runs = {"delilorn": measure_config(delilorn_config(sz, vocab, reps), vocab, T, B, toks),
+                "nekorax": measure_config(nekorax_like_delilorn_config(sz, vocab, n_layers), vocab, T, B, toks),
+                "veredra": measure_config(veredra_like_delilorn_config(sz, vocab, 2 * reps), vocab, T, B, toks)}
+
+        def frac(model, phases, per, prefill, decode):
+            """`prefill`, `decode`: (flops, bytes) of the phases in one layer; `per`: layers that have them."""
+            res = {}
+            for step, (flops, nbytes), key in (("prefill", prefill, "prefill"), ("decode", decode, "decode_per_step")):
+                ms = sum(runs[model]["phases_ms"][key].get(n, 0) for n in phases) / per
+                res[step] = None if not ms else round(max(flops / tf, nbytes / bw) / (ms / 1e3), 4)
+            return res
+
+        ctx, row = T - 64, kr + lr
+        seen = lambda k: sum(min(t + 1, win + k) for t in range(T))
+        att = lambda k: ((4.0 * D * H * seen(k), 0.0), (0.0, B * min(ctx, win + k) * G * 2 * D * 2.0))
+        lat = ((2.0 * lh * (T * (T + 1) // 2) * (row + kr), 0.0), (2.0 * B * lh * ctx * (row + kr), B * ctx * row * 2.0))
+        a_proj = (2 * H + 2 * G) * D * W
+        l_own, l_read = row * W, qr * W + qr * lh * (ld + lr) + lh * ld * kr + lh * kr * lv + lh * lv * W
+        n_proj = (2 * nh * nk + 3 * nh * nv) * W
+        proj = lambda n: ((2.0 * T * n, 0.0), (0.0, 2.0 * n))
+        rows = lambda nbytes: ((0.0, T * nbytes), (0.0, B * nbytes))
+        touched = E * (1.0 - (1.0 - top / E) ** B)
+        moe = lambda mats: ((2.0 * T * mats * W * top * eff, 0.0), (0.0, 2.0 * touched * mats * W * eff))
+        # q, k, v in and o out (and, for gated linear attention, a decay per key element)
+        scan = lambda decays: ((0.0, T * nh * (2 * nk + 2 * nv + decays * nk) * 4.0), (0.0, B * nh * nk * nv * 8.0))
+        latent_rows = lh * (ld + lr) * (4.0 + 2.0)
+        norms = W * ((4 + 4 + 4 + 2.0) + (top * 4 + 4 + 4 + 2.0))
+        roof = {
+            "attention over the cached latent": {
+                "delilorn": frac("delilorn", ["latent_attention"], 2 * reps, *lat), "nekorax": frac("nekorax", ["latent_attention"], n_layers, *lat)},
+            "windowed attention (with kept first tokens / without)": {
+                "delilorn": frac("delilorn", ["attention"], reps, *att(keep)), "veredra": frac("veredra", ["attention"], 2 * reps, *att(0))},
+            "recurrence (a constant decay per head / a decay per key element)": {
+                "delilorn": frac("delilorn", ["scan"], reps, *scan(0)), "veredra": frac("veredra", ["scan"], 2 * reps, *scan(1))},
+            "norm and gate after the recurrence": {
+                "delilorn": frac("delilorn", ["gated_norm"], reps, *rows(nh * nv * (4 + 4 + 2.0))),
+                "veredra": frac("veredra", ["gated_norm"], 2 * reps, *rows(nh * nv * (4 + 4 + 2.0)))},
+            "mixer projections in and out (all mixers of the model)": {
+                "delilorn": frac("delilorn", ["qkv", "wo"], reps, *proj(a_proj + n_proj + l_own + 2 * (l_read + lh * lv * W))),
+                "nekorax": frac("nekorax", ["qkv", "wo"], n_layers, *proj(l_own + l_read)),
+                "veredra": frac("veredra", ["qkv", "wo"], 2 * reps, *proj(a_proj + n_proj + 16 * W + 16 * nh * nk))},
+            "row kernels of the mixers (rotations, cache writes, gates)": {
+                "delilorn": frac("delilorn", ["kv_store", "head_post"], reps,
+                                 *rows((H + 2 * G) * D * (4 + 2.0) + 2 * (latent_rows + lh * lv * (2 + 2 + 4.0)) + row * (4 + 2.0))),
+                "nekorax": frac("nekorax", ["kv_store"], n_layers, *rows(latent_rows + row * (4 + 2.0))),
+                "veredra": frac("veredra", ["kv_store"], 2 * reps, *rows((H + 2 * G) * D * (4 + 2.0)))},
+            "routed experts with the router (two matrices / three)": {
+                "delilorn": frac("delilorn", ["moe_router", "moe_expert"], n_layers, *moe(2.0)),
+                "nekorax": frac("nekorax", ["moe_router", "moe_expert"], n_layers, *moe(3.0))},
+            "norms and the residual (the experts' sum, four norms and two sums in two kernels; the query latents' norms)": {
+                "delilorn": frac("delilorn", ["rmsnorm"], n_layers, *rows(norms + qr * (4 + 2.0) / 2)),
+                "nekorax": frac("nekorax", ["rmsnorm"], n_layers, *rows(norms + qr * (4 + 2.0)))},
+        }
+        out["points"][name] = {"sizes": sz, "layers": n_layers, "prefill_tokens": T, "decode_batch": B, "decode_context": ctx,
+                               **runs, "fraction_of_roofline": roof}
+    big = out["points"][sorted(out["points"])[-1]]
+    out["value"] = big["delilorn"]["decode_tok_s"]
+    out["config"] = {"model": "Delilorn: latent attention, lightning, latent attention over the same latent, windowed attention; routed experts",
+                     "global_batch": B, "seq_len": T, "parallelism": "single GPU", "l2": "weights of a step exceed the L2"}
+    return out
+
+
 def reference_arm_reason() -> str:
     """Why `--impl reference` has nothing to run, as found on this image (one line)."""
     return ("kurulav1/cpi is a CMake C++/CUDA project (no setup.py or pyproject.toml, so pip has nothing to install); "
@@ -1278,9 +1423,9 @@ def main() -> int:
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--context", type=int, default=4096)
     ap.add_argument("--skip-points", action="store_true")
-    ap.add_argument("--sizes", default="", help="--workload nogapel | kikerax | nekorax: a comma-separated subset of its size points")
+    ap.add_argument("--sizes", default="", help="--workload nogapel | kikerax | nekorax | delilorn: a comma-separated subset of its size points")
     ap.add_argument("--workload", choices=["scout24", "maverick4", "long131k", "contexts", "cpu_baseline", "veredra", "savenex", "nogapel", "kikerax",
-                                               "nekorax"],
+                                               "nekorax", "delilorn"],
                     default="scout24")
     ap.add_argument("--reference-root", default=os.environ.get("CPI_REFERENCE_ROOT"),
                     help="a checkout of kurulav1/cpi (for --workload cpu_baseline)")
@@ -1306,6 +1451,9 @@ def main() -> int:
         return 0
     if args.workload == "nekorax":
         print(json.dumps(run_nekorax(args)))
+        return 0
+    if args.workload == "delilorn":
+        print(json.dumps(run_delilorn(args)))
         return 0
     if args.workload == "nogapel":
         print(json.dumps(run_nogapel(args)))

@@ -764,11 +764,32 @@ def linear_scan(k, q, v, state, out, batch, *, n_heads, heads_per_group, n_rows,
     launch_count += 2 if run_len else 0
 
 
-def silu_rows(x):
-    """x <- silu(x) in place: float32 rows (a column slice allowed)."""
-    _need_cuda(x)
-    assert x.dtype == torch.float32 and x.dim() == 2 and x.stride(1) == 1
-    _call("cpi_silu_rows", _p(x), c_long(x.stride(0)), c_int(x.shape[0]), c_int(x.shape[1]), _stream())
+def silu_rows(x, out=None):
+    """out = silu(x) over float32 rows (a column slice allowed); out float32 or bfloat16, by default x itself."""
+    out = x if out is None else out
+    _need_cuda(x, out)
+    assert x.dtype == torch.float32 and x.dim() == 2 and x.stride(1) == 1 and out.shape == x.shape and out.stride(1) == 1
+    _call("cpi_silu_rows", _p(x), c_long(x.stride(0)), _p(out), c_int(dtype_code(out.dtype)), c_long(out.stride(0)),
+          c_int(x.shape[0]), c_int(x.shape[1]), _stream())
+
+
+def lightning_chunks_supported(n_rows, n_cols) -> bool:
+    return bool(load().cpi_lightning_chunks_supported(c_int(int(n_rows)), c_int(int(n_cols))))
+
+
+def lightning_chunks(qkv, decay, state, out, batch, *, n_heads, n_rows, n_cols):
+    """`linear_scan` with constant decays for bfloat16 rows qkv [T, heads * (2 n_rows + n_cols)] = [q | k | v] (their
+    activation done), in chunks on the tensor cores: out float32 [T, heads * n_cols], state float32 [slots, heads, n_rows,
+    n_cols] updated in place, decay float32 [heads].  For the sizes that `lightning_chunks_supported` takes."""
+    _need_cuda(qkv, decay, state, out)
+    T = qkv.shape[0]
+    assert qkv.dtype == torch.bfloat16 and qkv.stride(1) == 1 and qkv.shape[1] == n_heads * (2 * n_rows + n_cols)
+    assert decay.dtype == out.dtype == state.dtype == torch.float32 and decay.is_contiguous() and decay.numel() == n_heads
+    assert out.shape == (T, n_heads * n_cols) and out.stride(1) == 1
+    assert state.is_contiguous() and tuple(state.shape[1:]) == (n_heads, n_rows, n_cols)
+    _call("cpi_lightning_chunks", _p(qkv), c_long(qkv.stride(0)), _p(decay), _p(state), _p(out), c_long(out.stride(0)),
+          _p(batch.seq_slot), _p(batch.seq_tok0), _p(batch.seq_new), c_int(batch.n_seqs), c_int(n_heads), c_int(n_rows),
+          c_int(n_cols), _stream())
 
 
 def row_decay(z, z_bias, tau, *, kind=0, a_log=None, rows_per_head=0):

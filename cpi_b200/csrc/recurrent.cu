@@ -20,7 +20,9 @@
 //                      tokens are, a long prompt of this flavour is cut into runs that are scanned side by side: every
 //                      run from a zero state for what it adds (no outputs), the runs' entry states by one pass over
 //                      them (scan_chain), and every run again from its true entry state for the outputs.
-//   silu_rows          rows made silu(row) in place: what a prompt's recurrence would otherwise redo per block of columns.
+//                      (A bfloat16 prompt of this flavour goes through lightning.cu instead.)
+//   silu_rows          silu of float32 rows, in place or into another buffer in either precision: what a prompt's
+//                      recurrence would otherwise redo per block of columns.
 //   rglru_scan         a gated linear recurrent unit with one state element per channel (see its own comment);
 //   block_major_rows   the equal parts of float32 rows laid out part by part, as the rows of a grouped product.
 //   head_unit          rows of heads made unit vectors in place: x / sqrt(sum(x^2) + eps) per head.
@@ -478,18 +480,25 @@ __global__ void __launch_bounds__(128) head_unit_kernel(float* x, long stride, i
 }
 
 
-// z <- silu(z) over n columns of float32 rows, in place
-__global__ void __launch_bounds__(256) silu_rows_kernel(float* x, long stride, int n, int vec) {
+// out = silu(x) over n columns of float32 rows (out may be x); V columns a thread
+template <int V, typename TO>
+__global__ void __launch_bounds__(256) silu_rows_kernel(const float* x, long stride, TO* out, long out_stride, int n) {
   // (no early launch of the recurrence behind it: see row_decay_kernel)
   pdl_wait();
-  float* r = x + (size_t)blockIdx.x * stride;
-  const int i = blockIdx.y * blockDim.x + threadIdx.x;
-  if (vec) {
-    if (4 * i >= n) return;
-    float4 v = reinterpret_cast<float4*>(r)[i];
-    reinterpret_cast<float4*>(r)[i] = make_float4(silu_f(v.x), silu_f(v.y), silu_f(v.z), silu_f(v.w));
-  } else if (i < n) {
-    r[i] = silu_f(r[i]);
+  const int i = V * (blockIdx.y * blockDim.x + threadIdx.x);
+  if (i >= n) return;
+  const float* r = x + (size_t)blockIdx.x * stride + i;
+  TO* o = out + (size_t)blockIdx.x * out_stride + i;
+  if constexpr (V == 4) {
+    const float4 v = *reinterpret_cast<const float4*>(r);
+    if constexpr (sizeof(TO) == 4) {
+      *reinterpret_cast<float4*>(o) = make_float4(silu_f(v.x), silu_f(v.y), silu_f(v.z), silu_f(v.w));
+    } else {
+      __nv_bfloat162 a = __floats2bfloat162_rn(silu_f(v.x), silu_f(v.y)), b = __floats2bfloat162_rn(silu_f(v.z), silu_f(v.w));
+      *reinterpret_cast<uint2*>(o) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+    }
+  } else {
+    *o = from_f32<TO>(silu_f(*r));
   }
 }
 
@@ -801,11 +810,16 @@ extern "C" int cpi_linear_scan(const float* k, long k_stride, const float* q, lo
   return z ? dispatch_scan<kRowDecay>(p, n_seqs, max_new, stream) : dispatch_scan<kStepDecay>(p, n_seqs, max_new, stream);
 }
 
-extern "C" int cpi_silu_rows(float* x, long stride, int n_rows, int n, cudaStream_t stream) {
+extern "C" int cpi_silu_rows(const float* x, long stride, void* out, int out_dtype, long out_stride, int n_rows, int n,
+                             cudaStream_t stream) {
   if (n_rows == 0 || n == 0) return 0;
-  const int vec = (reinterpret_cast<uintptr_t>(x) & 15) == 0 && stride % 4 == 0 && n % 4 == 0;
-  const int items = vec ? n / 4 : n;
-  cpi::launch_pdl(silu_rows_kernel, dim3(n_rows, (items + 255) / 256), dim3(256), 0, stream, x, stride, n, vec);
+  const bool vec = ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out)) & 15) == 0 && stride % 4 == 0 &&
+                   out_stride % 4 == 0 && n % 4 == 0;
+  const dim3 grid(n_rows, ((vec ? n / 4 : n) + 255) / 256);
+  CPI_DISPATCH_DTYPE(out_dtype, TO, {
+    if (vec) cpi::launch_pdl(silu_rows_kernel<4, TO>, grid, dim3(256), 0, stream, x, stride, reinterpret_cast<TO*>(out), out_stride, n);
+    else cpi::launch_pdl(silu_rows_kernel<1, TO>, grid, dim3(256), 0, stream, x, stride, reinterpret_cast<TO*>(out), out_stride, n);
+  });
   return check_launch("silu_rows");
 }
 

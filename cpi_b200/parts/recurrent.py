@@ -37,6 +37,8 @@ from .linear import MODE_ADD, MODE_STORE, project
 
 # steps whose longest portion has more tokens than this prepare the row decays with a kernel of their own
 DECAY_PREPASS_FROM = 16
+# set to False to run every recurrence with constant decays token by token (tests compare the two)
+use_chunked_kernel = True
 # a recurrence with constant decays is cut into runs of at least this many tokens, until its blocks fill the GPU this often
 RUN_TOKENS = 64
 RUN_BLOCKS_PER_SM = 4
@@ -300,8 +302,10 @@ class LightningMixer(Mixer):
     tensor_names {"q", "k", "v", "g", "o", "norm"}.
     state: "s" [heads, key_dim, value_dim] float32.  The projections feed the recurrence as float32 rows.
 
-    A decode step's recurrence applies silu itself; a prompt's rows pass it once beforehand.  A long prompt of few
-    sequences is cut into runs that are scanned side by side (`csrc/recurrent.cu`: the runs of `linear_scan`)."""
+    A decode step's recurrence applies silu itself; a prompt's rows pass it once beforehand.  In bfloat16 a prompt's q, k
+    and v are rounded after silu and the recurrence runs in chunks on the tensor cores (`csrc/lightning.cu`); in float32,
+    and for sizes which that does not take, a long prompt of few sequences is cut into runs that are scanned side by side
+    (`csrc/recurrent.cu`: the runs of `linear_scan`)."""
     graph_safe = True
     can_store = True
 
@@ -356,16 +360,21 @@ class LightningMixer(Mixer):
             project(h, self.w_in, proj)
         o = self.ws.get("lightning_o", (T, nv), f32)
         with phase("scan"):
+            qkv, size = proj[:, :2 * nk + nv], dict(n_heads=self.nh, n_rows=self.dk, n_cols=self.dv)
             ready = batch.max_new > DECAY_PREPASS_FROM
-            if ready:
-                K.silu_rows(proj[:, :2 * nk + nv])
-            run_len, run_state = self.run_length(batch.n_seqs, batch.max_new), None
-            if run_len:
-                runs = -(-batch.max_new // run_len)
-                run_state = self.ws.get("lightning_runs", (batch.n_seqs * runs, nv * self.dk), f32)
-            K.linear_scan(proj[:, nk:2 * nk], proj[:, :nk], proj[:, 2 * nk:2 * nk + nv], cache.state("s"), o, batch,
-                          n_heads=self.nh, heads_per_group=1, n_rows=self.dk, n_cols=self.dv, decay=self.decay,
-                          silu=not ready, run_state=run_state, run_len=run_len)
+            if ready and use_chunked_kernel and h.dtype == torch.bfloat16 and K.lightning_chunks_supported(self.dk, self.dv):
+                rows = self.ws.get("lightning_qkv", (T, 2 * nk + nv), torch.bfloat16)
+                K.silu_rows(qkv, rows)
+                K.lightning_chunks(rows, self.decay, cache.state("s"), o, batch, **size)
+            else:
+                if ready:
+                    K.silu_rows(qkv)
+                run_len, run_state = self.run_length(batch.n_seqs, batch.max_new), None
+                if run_len:
+                    runs = -(-batch.max_new // run_len)
+                    run_state = self.ws.get("lightning_runs", (batch.n_seqs * runs, nv * self.dk), f32)
+                K.linear_scan(qkv[:, nk:2 * nk], qkv[:, :nk], qkv[:, 2 * nk:], cache.state("s"), o, batch,
+                              heads_per_group=1, decay=self.decay, silu=not ready, run_state=run_state, run_len=run_len, **size)
         with phase("gated_norm"):
             g = self.ws.get("lightning_gated", (T, nv), h.dtype)
             K.gated_norm(o, proj[:, 2 * nk + nv:], self.w_norm, g, parts=1, gate_first=False, eps=self.eps,

@@ -126,10 +126,49 @@ def test_recurrence_with_constant_decays(H, D, Dv, run):
             assert torch.equal(state[1].cpu(), S0[1])
 
 
+@pytest.mark.parametrize("H,D,Dv", [(4, 128, 128), (8, 32, 16), (1, 8, 8), (3, 24, 40), (2, 16, 200), (40, 64, 128), (2, 120, 48), (6, 56, 72)])
+def test_chunked_recurrence_on_the_tensor_cores(H, D, Dv):
+    """The same recurrence from bfloat16 rows, in chunks: whole, in portions that end inside chunks (down to one token),
+    beside sequences that are shorter than a chunk and that end on one, from entry states that are not zero.  The state and
+    the outputs are as exact as float32 sums are."""
+    g = torch.Generator().manual_seed(D * 3 + Dv)
+    lens, T = (31, 64), 210
+    decay = torch.tensor([(0.999, 0.0, 1.0, 0.31, 0.95, 0.5, 0.99, 0.9995)[h % 8] for h in range(H)])
+    C = H * (2 * D + Dv)
+    rows = rn(g, T, C + 8, std=1.2).bfloat16()
+    other = [rn(g, n, C + 8, std=1.2).bfloat16() for n in lens]
+    S0 = rn(g, 4, H, D, Dv)
+
+    def plain(r, S):
+        n, x = r.shape[0], r.double()
+        return P.decayed_sum(x[:, :H * D].view(n, H, D), x[:, H * D:2 * H * D].view(n, H, D), x[:, 2 * H * D:C].view(n, H, Dv), decay, S)
+
+    (want, end), beside = plain(rows, S0[2]), [plain(r, S0[s]) for r, s in zip(other, (3, 0))]
+    assert K().lightning_chunks_supported(D, Dv) and not K().lightning_chunks_supported(D + 4, Dv)
+    close = lambda a, b: ((a.cpu().double() - b).abs().max() < 1e-5 * b.abs().max())
+    for cuts in ([T], [100, 1, 2, 70, 37], [64, 146]):
+        state, outs, at = S0.to(DEV).clone(), [], 0
+        for i, n in enumerate(cuts):
+            b = FakeBatch([3, 2, 0], [0, at, 0], [lens[0], n, lens[1]]) if i == 0 else FakeBatch([2], [at], [n])
+            x = (torch.cat([other[0], rows[:n], other[1]]) if i == 0 else rows[at:at + n]).to(DEV)[:, :C]
+            o = torch.empty(x.shape[0], H * Dv, device=DEV)
+            K().lightning_chunks(x, decay.to(DEV), state, o, b, n_heads=H, n_rows=D, n_cols=Dv)
+            if i == 0:
+                assert close(o[:lens[0]].view(-1, H, Dv), beside[0][0]) and close(o[-lens[1]:].view(-1, H, Dv), beside[1][0])
+                o = o[lens[0]:-lens[1]]
+            outs.append(o)
+            at += n
+        assert close(torch.cat(outs).view(T, H, Dv), want), cuts
+        assert close(state[2], end) and close(state[3], beside[0][1]) and close(state[0], beside[1][1])
+        assert torch.equal(state[1].cpu(), S0[1])
+
+
 @pytest.mark.parametrize("W,H,D,Dv,dtype", [(54, 3, 10, 14, "float32"), (64, 8, 32, 16, "bfloat16"), (128, 2, 64, 128, "bfloat16"),
                                             (40, 1, 1, 1, "float32")])
 def test_lightning_mixer_alone(W, H, D, Dv, dtype):
-    """Projections, recurrence, the norm over all heads together, gate and output; runs on and off give the same rows."""
+    """Projections, recurrence, the norm over all heads together, gate and output; with the chunked kernel (bfloat16), in
+    runs, and token by token."""
+    from cpi_b200.parts import recurrent as R
     g = torch.Generator().manual_seed(W + D)
     dt = getattr(torch, dtype)
     T = 300
@@ -150,17 +189,21 @@ def test_lightning_mixer_alone(W, H, D, Dv, dtype):
 
     tol = 2e-5 if dtype == "float32" else 2e-2
     assert part.run_length(1, T) > 0 and part.run_length(1, 1) == 0
-    for runs in (True, False):
+    for how in ("chunks", "runs", "tokens"):
         cache, out, at = Cache(), [], 0
-        if not runs:
+        R.use_chunked_kernel = how == "chunks"
+        if how == "tokens":
             part.run_length = lambda n, t: 0
-        for n in (260, 2, 1, 37):
-            o = torch.empty(n, W, device=DEV)
-            part.forward(h[at:at + n].to(DEV), o, FakeBatch([0], [at], [n]), cache, add=False)
-            out.append(o)
-            at += n
+        try:
+            for n in (260, 2, 1, 37):
+                o = torch.empty(n, W, device=DEV)
+                part.forward(h[at:at + n].to(DEV), o, FakeBatch([0], [at], [n]), cache, add=False)
+                out.append(o)
+                at += n
+        finally:
+            R.use_chunked_kernel = True
         d = (torch.cat(out).cpu().double() - want).abs().max()
-        assert d < tol * want.abs().max(), runs
+        assert d < tol * want.abs().max(), how
 
 
 @pytest.mark.parametrize("H,G,D,Dv,dims", [(4, 2, 64, 64, 32), (8, 8, 128, 128, 64), (6, 2, 10, 14, 6), (2, 1, 128, 128, 128), (3, 1, 24, 16, 8),
@@ -434,13 +477,13 @@ def test_a_far_token_among_hundreds_and_long_decoding(models, name):
 
 
 def test_fused_and_separate_kernels_agree(models):
-    """The fused preparation and the tensor-core attention kernels, and the separate and general ones, in bfloat16: both
-    give the plain implementation's logits (with the choices of experts that each of them made)."""
-    from cpi_b200.parts import attention as A
+    """The fused preparation, the tensor-core attention kernels and the chunked recurrence, and the separate and general
+    ones, in bfloat16: both give the plain implementation's logits (with the choices of experts that each of them made)."""
+    from cpi_b200.parts import attention as A, recurrent as R
     b = models["B"]
     toks = V.tokens(300, b.cfg["vocab"], 3)
     for on in (True, False):
-        A.use_tensor_core_kernels = A.use_fused_preparation = on
+        A.use_tensor_core_kernels = A.use_fused_preparation = R.use_chunked_kernel = on
         try:
             r = Run(b.engine("bfloat16", max_tokens=1024, max_seqs=2))
             r.step([("x", toks[:200], range(0, 200, 7))])
@@ -449,7 +492,7 @@ def test_fused_and_separate_kernels_agree(models):
                 r.step([("x", toks[i:i + 1], [0])])
             r.check(b, {"x": toks}, TOL["bfloat16"])
         finally:
-            A.use_tensor_core_kernels = A.use_fused_preparation = True
+            A.use_tensor_core_kernels = A.use_fused_preparation = R.use_chunked_kernel = True
 
 
 def test_other_constants_change_the_result_as_the_plain_implementation_says(tmp_path):
