@@ -689,6 +689,12 @@ def measure_config(cfg, vocab, T, B, toks):
     res["decode_ms_per_step"] = round(e0.elapsed_time(e1) / 32, 4)
     res["decode_tok_s"] = round(B / (res["decode_ms_per_step"] / 1e3), 1)
     res["graphs"] = bool(eng.use_graphs)
+    chosen = eng.capture_routing(True)          # distinct experts per routed layer that a decode step's tokens choose
+    eng.step([StepEntry(s, toks(1), [0]) for s in slots])
+    counts = [len(set(x.flatten().tolist())) for lst in chosen.values() for x in lst]
+    eng.capture_routing(False)
+    if counts:
+        res["experts_touched_per_decode_step"] = round(sum(counts) / len(counts), 2)
     timer = eng.profile_phases(True)
     for _ in range(4):
         eng.step([StepEntry(s, toks(1), [0]) for s in slots])
@@ -1363,8 +1369,8 @@ def run_delilorn(args) -> dict:
         n_proj = (2 * nh * nk + 3 * nh * nv) * W
         proj = lambda n: ((2.0 * T * n, 0.0), (0.0, 2.0 * n))
         rows = lambda nbytes: ((0.0, T * nbytes), (0.0, B * nbytes))
-        touched = E * (1.0 - (1.0 - top / E) ** B)
-        moe = lambda mats: ((2.0 * T * mats * W * top * eff, 0.0), (0.0, 2.0 * touched * mats * W * eff))
+        touched = lambda m: runs[m]["experts_touched_per_decode_step"]
+        moe = lambda m, mats: ((2.0 * T * mats * W * top * eff, 0.0), (0.0, 2.0 * touched(m) * mats * W * eff))
         # q, k, v in and o out (and, for gated linear attention, a decay per key element)
         scan = lambda decays: ((0.0, T * nh * (2 * nk + 2 * nv + decays * nk) * 4.0), (0.0, B * nh * nk * nv * 8.0))
         latent_rows = lh * (ld + lr) * (4.0 + 2.0)
@@ -1389,8 +1395,8 @@ def run_delilorn(args) -> dict:
                 "nekorax": frac("nekorax", ["kv_store"], n_layers, *rows(latent_rows + row * (4 + 2.0))),
                 "veredra": frac("veredra", ["kv_store"], 2 * reps, *rows((H + 2 * G) * D * (4 + 2.0)))},
             "routed experts with the router (two matrices / three)": {
-                "delilorn": frac("delilorn", ["moe_router", "moe_expert"], n_layers, *moe(2.0)),
-                "nekorax": frac("nekorax", ["moe_router", "moe_expert"], n_layers, *moe(3.0))},
+                "delilorn": frac("delilorn", ["moe_router", "moe_expert"], n_layers, *moe("delilorn", 2.0)),
+                "nekorax": frac("nekorax", ["moe_router", "moe_expert"], n_layers, *moe("nekorax", 3.0))},
             "norms and the residual (the experts' sum, four norms and two sums in two kernels; the query latents' norms)": {
                 "delilorn": frac("delilorn", ["rmsnorm"], n_layers, *rows(norms + qr * (4 + 2.0) / 2)),
                 "nekorax": frac("nekorax", ["rmsnorm"], n_layers, *rows(norms + qr * (4 + 2.0)))},

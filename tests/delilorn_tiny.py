@@ -170,6 +170,14 @@ def draw_weights(cfg: dict, seed: int) -> dict:
     return W
 
 
+def strong_sublayers(W: dict) -> None:
+    """Weights under which a greedy continuation moves about: with the output matrix being the embedding table, a residual
+    in which the token's own embedding dominates would predict that token again and again."""
+    for name in W:
+        if name.endswith((".norm1b", ".norm2b")):
+            W[name] = W[name] + 4.0
+
+
 def write_model(cfg: dict, W: dict, root=None) -> str:
     from cpi_b200.weights.safetensors_io import write_safetensors
     d = tempfile.mkdtemp(prefix="delilorn_tiny_", dir=root)
