@@ -466,6 +466,60 @@ __global__ void __launch_bounds__(128) gated_norm_kernel(GatedNormParams p) {
   }
 }
 
+// The same for wide parts (1,024 elements or more, whole groups of four on 16 bytes, a float32 weight per element of a part
+// or of the row): four elements a thread at a time, kept in registers between the two passes.  The block's size follows from the width of a part alone.
+constexpr int GN_THREADS = 512, GN_PER = 4;
+template <typename TO>
+__global__ void __launch_bounds__(GN_THREADS) gated_norm_wide_kernel(GatedNormParams p) {
+  pdl_launch_dependents();
+  __shared__ float scratch[32];
+  const int t = blockIdx.x, part = blockIdx.y, n = p.width / p.parts, groups = n >> 2;
+  const float4* y = reinterpret_cast<const float4*>(p.y + (size_t)t * p.y_stride + (size_t)part * n);
+  const float4* g = p.gate ? reinterpret_cast<const float4*>(p.gate + (size_t)t * p.gate_stride + (size_t)part * n) : nullptr;
+  const float4* w = p.w ? reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.w) + (p.w_len == n ? 0 : part * n)) : nullptr;
+  float4 v[GN_PER], a[GN_PER], wt[GN_PER];
+#pragma unroll
+  for (int j = 0; j < GN_PER; ++j) {                         // no kernel writes the weight
+    const int i = threadIdx.x + j * blockDim.x;
+    wt[j] = w && i < groups ? w[i] : make_float4(1.f, 1.f, 1.f, 1.f);
+  }
+  pdl_wait();
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < GN_PER; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    a[j] = make_float4(1.f, 1.f, 1.f, 1.f);
+    if (i >= groups) continue;
+    v[j] = y[i];
+    if (g) a[j] = g[i];
+  }
+#pragma unroll
+  for (int j = 0; j < GN_PER; ++j) {
+    if (g) a[j] = make_float4(gate_f(a[j].x, p.gate_act), gate_f(a[j].y, p.gate_act), gate_f(a[j].z, p.gate_act), gate_f(a[j].w, p.gate_act));
+    if (p.gate_first) {
+      v[j] = make_float4(v[j].x * a[j].x, v[j].y * a[j].y, v[j].z * a[j].z, v[j].w * a[j].w);
+      a[j] = make_float4(1.f, 1.f, 1.f, 1.f);
+    }
+    ss = fmaf(v[j].x, v[j].x, fmaf(v[j].y, v[j].y, fmaf(v[j].z, v[j].z, fmaf(v[j].w, v[j].w, ss))));
+  }
+  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)n + p.eps);
+  TO* o = reinterpret_cast<TO*>(p.out) + (size_t)t * p.out_stride + (size_t)part * n;
+#pragma unroll
+  for (int j = 0; j < GN_PER; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i >= groups) continue;
+    const float r[4] = {v[j].x * inv * wt[j].x * a[j].x, v[j].y * inv * wt[j].y * a[j].y, v[j].z * inv * wt[j].z * a[j].z,
+                        v[j].w * inv * wt[j].w * a[j].w};
+    if constexpr (sizeof(TO) == 4) {
+      *reinterpret_cast<float4*>(o + 4 * i) = make_float4(r[0], r[1], r[2], r[3]);
+    } else {
+      __nv_bfloat162 lo = __floats2bfloat162_rn(r[0], r[1]), hi = __floats2bfloat162_rn(r[2], r[3]);
+      *reinterpret_cast<uint2*>(o + 4 * i) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+    }
+  }
+}
+
 // x[t, head, :] <- x / sqrt(sum(x^2) + eps) in place, float32 rows of `heads` heads of `dim` elements; a warp per head
 __global__ void __launch_bounds__(128) head_unit_kernel(float* x, long stride, int heads, int dim, float eps) {
   pdl_launch_dependents();
@@ -842,6 +896,15 @@ extern "C" int cpi_gated_norm(const float* y, long y_stride, const float* gate, 
   CPI_REQUIRE(!w || w_len > 0, "gated_norm: a weight needs a length");
   CPI_REQUIRE(gate_act == 0 || gate_act == 1, "gated_norm: unknown gate activation %d", gate_act);
   GatedNormParams p{y, y_stride, gate, gate_stride, w, w_dtype, w_len, out, out_stride, width, parts, gate_first, eps, gate_act};
+  const int n = width / parts;
+  auto ok16 = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  if (n >= 1024 && n % 4 == 0 && n <= 4 * GN_PER * GN_THREADS && ok16(y) && ok16(gate) && ok16(out) && ok16(w) &&
+      (!w || (w_dtype == kF32 && (w_len == n || w_len == width))) && y_stride % 4 == 0 &&
+      gate_stride % 4 == 0 && out_stride % 4 == 0) {
+    const int threads = n <= 2048 ? 256 : GN_THREADS;
+    CPI_DISPATCH_DTYPE(out_dtype, TO, cpi::launch_pdl(gated_norm_wide_kernel<TO>, dim3(n_tokens, parts), dim3(threads), 0, stream, p));
+    return check_launch("gated_norm");
+  }
   CPI_DISPATCH_DTYPE(out_dtype, TO, cpi::launch_pdl(gated_norm_kernel<TO>, dim3(n_tokens, parts), 128, 0, stream, p));
   return check_launch("gated_norm");
 }

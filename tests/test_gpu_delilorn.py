@@ -206,7 +206,28 @@ def test_lightning_mixer_alone(W, H, D, Dv, dtype):
         assert d < tol * want.abs().max(), how
 
 
-@pytest.mark.parametrize("H,G,D,Dv,dims", [(4, 2, 64, 64, 32), (8, 8, 128, 128, 64), (6, 2, 10, 14, 6), (2, 1, 128, 128, 128), (3, 1, 24, 16, 8),
+@pytest.mark.parametrize("W,parts", [(54, 1), (1000, 1), (1024, 1), (1028, 1), (2052, 1), (4096, 1), (8192, 1), (8196, 1), (4096, 4), (3072, 2), (6, 3)])
+def test_norm_and_gate_over_rows_of_several_widths(W, parts):
+    """The norm that follows the recurrence, gate after it and before it, silu and sigmoid, one weight per element or shared
+    by the parts: narrow rows and wide ones, which take a kernel of their own, gates that are a slice of wider rows."""
+    g = torch.Generator().manual_seed(W)
+    T, eps, n = 5, 1e-2, W // parts
+    y, gate = rn(g, T, W, std=0.3), rn(g, T, W + 8, std=2.0)
+    for wlen in {W, n}:
+        w = rn(g, wlen, std=0.3, mean=1.0)
+        full = w.double().repeat(W // wlen)
+        for act, f in (("sigmoid", torch.sigmoid), ("silu", P.silu)):
+            a = f(gate[:, 8:].double())
+            for first in (False, True):
+                v = y.double() * a if first else y.double()
+                want = P.rms(v.view(T, parts, n), eps).reshape(T, W) * full * (1.0 if first else a)
+                for dt, tol in ((torch.float32, 3e-6), (torch.bfloat16, 6e-3)):
+                    out = torch.empty(T, W, dtype=dt, device=DEV)
+                    K().gated_norm(y.to(DEV), gate.to(DEV)[:, 8:], w.to(DEV), out, parts=parts, gate_first=first, eps=eps, gate_act=act)
+                    assert (out.cpu().double() - want).abs().max() < tol * want.abs().max(), (act, first, dt)
+
+
+@pytest.mark.parametrize("H,G,D,Dv,dims", [(4, 2, 64, 64, 32), (8, 4, 128, 128, 96), (6, 2, 10, 14, 6), (2, 1, 128, 128, 128), (3, 1, 24, 16, 8),
                                            (2, 2, 16, 40, 0), (5, 1, 8, 8, 8)])
 def test_rotation_of_part_of_a_head_into_the_pages(H, G, D, Dv, dims):
     """Queries turned, keys turned and values as they are into the pages of their positions: the fused kernel without a
